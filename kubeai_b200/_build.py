@@ -37,6 +37,7 @@ SOURCES = [
     "zinavik.cu",
     "mulenex.cu",
     "nagilix.cu",
+    "soselix.cu",
     "model_registry.cc",
     "abi_ops.cu",
     "engine.cu",

@@ -15,6 +15,11 @@
 // matrix memory with exponential gating (mLSTM): its gates come from `mlstm_gates`, its normaliser n_t = d n + s k and the
 // product n . q ride along in the scan's first column block (GlaArgs::nstate / nq), and `recurrent_out_gate` divides by
 // max(|n . q|, exp(-m)) before the norm.
+//
+// Two more forms are variants of the staging pass only.  HGRN2 (fgate_lower): the key columns hold forget-gate
+// pre-activations; the pass turns each into the channel's decay f = l + (1 - l) sigmoid(g) and the key 1 - f, so neither is
+// ever written to memory.  Mamba-2 (dt_pre): the decay exp(rate d) and the key scale d = softplus(dt + bias) of a
+// (token, head) are formed there, and the heads of a group read one key and query row (group).
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 
@@ -33,6 +38,7 @@ __device__ __forceinline__ float ldf(const bf16* p) { return __bfloat162float(__
 __device__ __forceinline__ void stf(float* p, float v) { *p = v; }
 __device__ __forceinline__ void stf(bf16* p, float v) { *p = __float2bfloat16_rn(v); }
 __device__ __forceinline__ float siluf_(float x) { return x / (1.0f + expf(-x)); }
+__device__ __forceinline__ float softplusf_(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
 
 constexpr int kRows = 32;      // key rows of the state held by one thread
 constexpr int kGroup = 16;     // tokens staged per shared-memory round (fewer when dim is large)
@@ -61,6 +67,9 @@ __global__ void gla_decay_kernel(float* z, const float* bias, int HD, float inv_
 // decay row is staged or read, the constant sits in a register.  MODE 2: one decay and one key scale per (token, head)
 // (GlaArgs::tok_decay / tok_kscale): both sit in shared memory as G scalars per round; the key scale multiplies the token's
 // value (and the normaliser's key) in the chain, (s k) v^T = k (s v)^T.
+// With GlaArgs::dt_pre the two scalars come from the step-size pre-activation as they are staged.
+// MODE 3: learned per-channel decays that also give the key (GlaArgs::fgate_lower), both formed from the pre-activation as it
+// is staged; one exponential serves the sigmoid and its complement, so 1 - f keeps its low bits where f is near 1.
 // NRM (with MODE 2): the CTAs of the first column block also carry the normaliser n [dim] of the head, n <- decay n + k
 // (what the scan does to a state column whose value is 1).  The threads of a row slice share its rows (thread jj owns rows
 // jj, jj + tcols, ... of the slice, at most kNormRows of them); every thread leaves its part of n . q in shared memory, and
@@ -69,7 +78,7 @@ __global__ void gla_decay_kernel(float* z, const float* bias, int HD, float inv_
 constexpr int kNormRows = 8;
 template <typename T, int NC, int MODE, int NE>
 __global__ void __launch_bounds__(kThreads) gla_scan_kernel(GlaArgs a, int P, int rpp, int G) {
-  constexpr bool CD = MODE != 0;
+  constexpr bool CD = MODE == 1 || MODE == 2;
   constexpr bool NRM = NE > 0;
   extern __shared__ __align__(16) float sm[];
   const int seq = blockIdx.z, head = blockIdx.y;
@@ -108,7 +117,8 @@ __global__ void __launch_bounds__(kThreads) gla_scan_kernel(GlaArgs a, int P, in
       S[c][r] = (live[c] && r < rpp && i < D && pos0 > 0) ? Sg[static_cast<long long>(i) * Dv + j[c]] : 0.f;
     }
   const int slice_elems = P * rpp;
-  const bool silu = a.act == GLA_ACT_SILU;
+  const bool silu = a.act == GLA_ACT_SILU, silu_q = silu || a.act == GLA_ACT_SILU_Q;
+  const int qk0 = (head / a.group) * D;   // the head's columns in the query and key blocks
   const float hdecay = MODE == 1 ? a.head_decay[head] : 0.f;
   for (int g0 = 0; g0 < n; g0 += G) {
     const int gn = min(G, n - g0);
@@ -117,14 +127,22 @@ __global__ void __launch_bounds__(kThreads) gla_scan_kernel(GlaArgs a, int P, in
     for (int x = threadIdx.x; x < slice_elems; x += kThreads) {
       const int pp = x / rpp, r = x - pp * rpp, i = pp * rpp + r;
       float* s3 = sm + pp * ps + r;
-      const int c = head * D + i;
+      const int c = qk0 + i;
       if (i < D) {
+        const float fb = MODE == 3 ? __ldg(a.z_bias + c) : 0.f, fl = MODE == 3 ? __ldg(a.fgate_lower + c) : 0.f;
 #pragma unroll 4
         for (int tt = 0; tt < gn; ++tt) {
           const long long row = static_cast<long long>(tok0 + g0 + tt);
           const T* rp = base + row * a.ld;
           float qv = ldf(rp + a.q_off + c), kv = ldf(rp + a.k_off + c);
-          if (silu) { qv = siluf_(qv); kv = siluf_(kv); }
+          if (silu_q) qv = siluf_(qv);
+          if (silu) kv = siluf_(kv);
+          if (MODE == 3) {
+            const float g = kv + fb, e = expf(-fabsf(g)), r = 1.0f / (1.0f + e), er = e * r;
+            const float hi = g >= 0.f ? r : er, lo = g >= 0.f ? er : r;     // sigmoid(g), sigmoid(-g)
+            s3[(tt * 3 + 2) * Dp] = fmaf(1.0f - fl, hi, fl);
+            kv = (1.0f - fl) * lo;
+          }
           if (a.rope && i < a.rot_dims) {
             // rotate-half layout: dimension i of the head is paired with i + rot_dims / 2
             const int half = a.rot_dims >> 1;
@@ -137,7 +155,7 @@ __global__ void __launch_bounds__(kThreads) gla_scan_kernel(GlaArgs a, int P, in
           }
           s3[(tt * 3) * Dp] = qv * a.q_scale;
           s3[(tt * 3 + 1) * Dp] = kv * a.k_scale;
-          if (!CD) s3[(tt * 3 + 2) * Dp] = __ldg(a.z + row * (a.heads * D) + c);
+          if (MODE == 0) s3[(tt * 3 + 2) * Dp] = __ldg(a.z + row * (a.heads * D) + c);
         }
       } else {
         for (int tt = 0; tt < gn; ++tt) { s3[(tt * 3) * Dp] = 0.f; s3[(tt * 3 + 1) * Dp] = 0.f; s3[(tt * 3 + 2) * Dp] = 0.f; }
@@ -151,8 +169,15 @@ __global__ void __launch_bounds__(kThreads) gla_scan_kernel(GlaArgs a, int P, in
     }
     if (MODE == 2)
       for (int tt = threadIdx.x; tt < gn; tt += kThreads) {
-        ds[tt] = __ldg(a.tok_decay + static_cast<long long>(tok0 + g0 + tt) * a.heads + head);
-        ds[G + tt] = __ldg(a.tok_kscale + static_cast<long long>(tok0 + g0 + tt) * a.heads + head);
+        const long long row = tok0 + g0 + tt;
+        if (a.dt_pre) {
+          const float d = softplusf_(ldf(static_cast<const T*>(a.dt_pre) + row * a.ld_dt + head) + __ldg(a.dt_bias + head));
+          ds[tt] = expf(__ldg(a.dt_rate + head) * d);
+          ds[G + tt] = d;
+        } else {
+          ds[tt] = __ldg(a.tok_decay + row * a.heads + head);
+          ds[G + tt] = __ldg(a.tok_kscale + row * a.heads + head);
+        }
       }
     __syncthreads();
     for (int tt = 0; tt < gn; ++tt) {
@@ -273,7 +298,7 @@ __global__ void recurrent_out_gate_kernel(OutGateArgs a, long long units) {
   const long long th = t * a.heads + c0 / a.vdim;
   const float dinv = a.den_nq ? 1.0f / (fmaxf(fabsf(a.den_nq[th]), a.den_floor[th]) + a.den_eps) : 1.0f;
   const float* w = a.w ? a.w + (a.w_full ? c0 : 0) : nullptr;   // null: a norm without a weight
-  const T* g = static_cast<const T*>(a.g) + t * a.ldg + c0;
+  const T* g = a.g ? static_cast<const T*>(a.g) + t * a.ldg + c0 : nullptr;
   T* y = static_cast<T*>(a.y) + t * a.ldy + c0;
   float ss = 0.f;
   for (int i = first; i < n; i += step) { const float v = op[i] * dinv; ss = fmaf(v, v, ss); }
@@ -286,10 +311,74 @@ __global__ void recurrent_out_gate_kernel(OutGateArgs a, long long units) {
   }
   const float inv = 1.0f / sqrtf(ss / static_cast<float>(n) + a.eps);
   for (int i = first; i < n; i += step) {
-    const float gv = ldf(g + i);
-    const float sg = 1.0f / (1.0f + expf(-gv));
-    const float gate = a.gate_act == GATE_SIGMOID ? sg : gv * sg;
+    float gate = 1.0f;
+    if (g) {
+      const float gv = ldf(g + i);
+      const float sg = 1.0f / (1.0f + expf(-gv));
+      gate = a.gate_act == GATE_SIGMOID ? sg : gv * sg;
+    }
     stf(y + i, op[i] * dinv * inv * (w ? w[i] : 1.0f) * gate * a.out_scale);
+  }
+}
+
+// The output stage with the gate in front of the norm (GatedGroupNormArgs): one CTA per (token, part).  VEC: four
+// neighbouring columns per thread and round (every part a whole number of fours inside a head).  The gated row stays in
+// shared memory between the two passes; the warps' sums of squares are added in warp order.
+__device__ __forceinline__ float4 ldf4(const float* p) { return __ldg(reinterpret_cast<const float4*>(p)); }
+__device__ __forceinline__ float4 ldf4(const bf16* p) {
+  const uint2 v = __ldg(reinterpret_cast<const uint2*>(p));
+  return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xffff0000u), __uint_as_float(v.y << 16), __uint_as_float(v.y & 0xffff0000u));
+}
+__device__ __forceinline__ void stf4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void stf4(bf16* p, float4 v) {
+  const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+  *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256) gated_group_norm_kernel(GatedGroupNormArgs a) {
+  extern __shared__ __align__(16) float us[];
+  __shared__ float red[8];
+  const long long t = blockIdx.x;
+  const int HV = a.heads * a.vdim, n = HV / a.groups, c0 = blockIdx.y * n;
+  const float* o = a.o + t * HV + c0;
+  const T* x = a.skip ? static_cast<const T*>(a.x) + t * a.ldx + c0 : nullptr;
+  const T* z = static_cast<const T*>(a.z) + t * a.ldz + c0;
+  constexpr int C = VEC ? 4 : 1;
+  float ss = 0.f;
+  for (int i = threadIdx.x * C; i < n; i += blockDim.x * C) {
+    float u[4], zv[4], xv[4] = {0.f, 0.f, 0.f, 0.f};
+    if (VEC) {
+      const float4 o4 = ldf4(o + i), z4 = ldf4(z + i);
+      u[0] = o4.x; u[1] = o4.y; u[2] = o4.z; u[3] = o4.w;
+      zv[0] = z4.x; zv[1] = z4.y; zv[2] = z4.z; zv[3] = z4.w;
+      if (x) { const float4 x4 = ldf4(x + i); xv[0] = x4.x; xv[1] = x4.y; xv[2] = x4.z; xv[3] = x4.w; }
+    } else {
+      u[0] = o[i]; zv[0] = ldf(z + i);
+      if (x) xv[0] = ldf(x + i);
+    }
+    const float d = x ? __ldg(a.skip + (c0 + i) / a.vdim) : 0.f;
+#pragma unroll
+    for (int c = 0; c < C; ++c) {
+      u[c] = fmaf(d, xv[c], u[c]) * siluf_(zv[c]);
+      us[i + c] = u[c];
+      ss = fmaf(u[c], u[c], ss);
+    }
+  }
+  for (int s = 16; s > 0; s >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, s);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+  __syncthreads();
+  ss = 0.f;
+  for (int w = 0; w < (blockDim.x >> 5); ++w) ss += red[w];
+  const float inv = 1.0f / sqrtf(ss / static_cast<float>(n) + a.eps);
+  const float* wt = a.w + c0;
+  T* y = static_cast<T*>(a.y) + t * a.ldy + c0;
+  for (int i = threadIdx.x * C; i < n; i += blockDim.x * C) {   // each thread reads back what it wrote
+    if (VEC) {
+      const float4 u = *reinterpret_cast<const float4*>(us + i), w = ldf4(wt + i);
+      stf4(y + i, make_float4(u.x * inv * w.x, u.y * inv * w.y, u.z * inv * w.z, u.w * inv * w.w));
+    } else {
+      stf(y + i, us[i] * inv * wt[i]);
+    }
   }
 }
 
@@ -343,10 +432,30 @@ int mlstm_gates(const MlstmGateArgs& a, cudaStream_t st) {
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
 
+int gated_group_norm(const GatedGroupNormArgs& a, cudaStream_t st) {
+  if (a.T <= 0) return 0;
+  if (!a.o || !a.z || !a.w || !a.y || a.heads < 1 || a.vdim < 1 || a.groups < 1 || (a.heads * a.vdim) % a.groups || (a.skip && !a.x)) return -1;
+  const int n = a.heads * a.vdim / a.groups;
+  const size_t smem = static_cast<size_t>(n) * sizeof(float);
+  if (smem > 47 * 1024) return -1;
+  auto al16 = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+  const bool vec = n % 4 == 0 && a.vdim % 4 == 0 && a.ldz % 4 == 0 && a.ldy % 4 == 0 && (!a.skip || a.ldx % 4 == 0) && al16(a.o) && al16(a.z) && al16(a.w) &&
+                   al16(a.y) && al16(a.x);
+  const int work = vec ? n / 4 : n;
+  const int th = work >= 256 ? 256 : (work >= 128 ? 128 : 64);
+  dim3 grid(a.T, a.groups);
+  if (a.t == DT_BF16) {
+    if (vec) gated_group_norm_kernel<bf16, true><<<grid, th, smem, st>>>(a); else gated_group_norm_kernel<bf16, false><<<grid, th, smem, st>>>(a);
+  } else {
+    if (vec) gated_group_norm_kernel<float, true><<<grid, th, smem, st>>>(a); else gated_group_norm_kernel<float, false><<<grid, th, smem, st>>>(a);
+  }
+  return cudaGetLastError() == cudaSuccess ? 0 : -2;
+}
+
 int recurrent_out_gate(const OutGateArgs& a, cudaStream_t st) {
   const long long units = a.joint ? a.T : static_cast<long long>(a.T) * a.heads;
   if (units <= 0) return 0;
-  if (!a.o || !a.g || !a.y || a.heads < 1 || a.vdim < 1) return -1;
+  if (!a.o || !a.y || a.heads < 1 || a.vdim < 1) return -1;
   if (a.joint && (a.w_full || a.den_nq)) return -1;
   if (a.den_nq && !a.den_floor) return -1;
   const int th = a.joint ? (a.heads * a.vdim >= 1024 ? 256 : 128) : 128;
@@ -381,9 +490,12 @@ int gla_scan(const GlaArgs& a, cudaStream_t st) {
   if (smem > 48 * 1024) return -1;
   if ((a.nstate != nullptr) != (a.nq != nullptr) || (a.nstate && !a.tok_decay)) return -1;
   if (a.nstate && rows_per_part > kNormRows * tcols) return -1;
+  if (a.group < 1 || a.heads % a.group || (a.group > 1 && !a.tok_decay && !a.dt_pre && !a.head_decay)) return -1;
+  if (a.dt_pre && (!a.dt_bias || !a.dt_rate || a.tok_decay || a.head_decay || a.fgate_lower || a.nstate)) return -1;
+  if (a.fgate_lower && (!a.z_bias || a.tok_decay || a.head_decay || a.rope || a.act == GLA_ACT_SILU)) return -1;
   if (a.tok_decay) {
     if (!a.tok_kscale || a.head_decay) return -1;
-  } else if (!a.head_decay) {
+  } else if (!a.head_decay && !a.dt_pre && !a.fgate_lower) {
     if (!a.z || !a.z_bias) return -1;
     const long long total = static_cast<long long>(a.T) * a.heads * a.dim;
     if (total > 0) gla_decay_kernel<<<static_cast<unsigned>((total + 255) / 256), 256, 0, st>>>(a.z, a.z_bias, a.heads * a.dim, a.inv_tau, total);
@@ -391,7 +503,8 @@ int gla_scan(const GlaArgs& a, cudaStream_t st) {
   const bool one_row = rows_per_part <= tcols;
 #define SCAN(T_, NC_) do { if (a.tok_decay && a.nstate && one_row) gla_scan_kernel<T_, NC_, 2, 1><<<grid, kThreads, smem, st>>>(a, P, rows_per_part, G); \
                           else if (a.tok_decay && a.nstate) gla_scan_kernel<T_, NC_, 2, kNormRows><<<grid, kThreads, smem, st>>>(a, P, rows_per_part, G); \
-                          else if (a.tok_decay) gla_scan_kernel<T_, NC_, 2, 0><<<grid, kThreads, smem, st>>>(a, P, rows_per_part, G); \
+                          else if (a.tok_decay || a.dt_pre) gla_scan_kernel<T_, NC_, 2, 0><<<grid, kThreads, smem, st>>>(a, P, rows_per_part, G); \
+                          else if (a.fgate_lower) gla_scan_kernel<T_, NC_, 3, 0><<<grid, kThreads, smem, st>>>(a, P, rows_per_part, G); \
                           else if (a.head_decay) gla_scan_kernel<T_, NC_, 1, 0><<<grid, kThreads, smem, st>>>(a, P, rows_per_part, G); \
                           else gla_scan_kernel<T_, NC_, 0, 0><<<grid, kThreads, smem, st>>>(a, P, rows_per_part, G); } while (0)
   if (a.t == DT_BF16) {

@@ -350,7 +350,7 @@ __global__ void __launch_bounds__(256) sandwich_step_kernel(SandwichArgs a) {
     else xv[0] = x[i];
     if (y) {
 #pragma unroll
-      for (int c = 0; c < C; ++c) xv[c] += a.post_w ? row[i + c] * inv_y * a.post_w[i + c] : row[i + c];   // each thread reads back what it wrote
+      for (int c = 0; c < C; ++c) xv[c] = fmaf(a.mult, a.post_w ? row[i + c] * inv_y * a.post_w[i + c] : row[i + c], xv[c]);   // each thread reads back what it wrote
       if (VEC) st4(x + i, make_float4(xv[0], xv[1], xv[2], xv[3]));
       else x[i] = xv[0];
     }

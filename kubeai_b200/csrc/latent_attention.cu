@@ -5,8 +5,11 @@
 // sum afterwards — so neither prefill nor decode ever rebuilds per-head keys or values of the window, and both read the
 // same paged cache rows [slot][kv_rank + rot_dim].  The two per-head projections are batched launches of linear.cu.
 //
-// Rotation: interleaved pairs (2i, 2i+1) of the first rot_dims of the rotated part, angles from a table computed in
-// double.  Window: key j is visible from position p when 0 <= p - j < window.  Softmax statistics are fp32.
+// Rotation: interleaved pairs (2i, 2i+1) of the first rot_dims of the rotated part, or pairs (i, i + rot_dims / 2); angles
+// from a table computed in double.  Window: key j is visible from position p when 0 <= p - j < window.  Softmax statistics
+// are fp32.  A sink is a score without a key: the running maximum starts at it and the running sum at 1, so the first tile
+// of keys already meets it.  In the split form only the first split starts that way.  The per-head output gate is applied
+// to the latent sum, ahead of W_uv (the two commute).
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <float.h>
@@ -51,50 +54,67 @@ __device__ __forceinline__ float block_max(float v, float* red) {
   return s;
 }
 
+// element i of a rotated row u: the pair it belongs to, its partner and its side (pairs at or past rot_dims / 2: unchanged)
+template <typename T>
+__device__ __forceinline__ float rotated(const T* u, int i, int half, bool half_pairs, const float2* cs) {
+  const float v = ldf(u + i);
+  if (i >= 2 * half) return v;
+  const bool high = half_pairs ? i >= half : (i & 1);
+  const int pr = half_pairs ? (high ? i - half : i) : i >> 1;
+  const float w = ldf(u + (half_pairs ? (high ? i - half : i + half) : i ^ 1));
+  const float2 c = cs[pr];
+  return high ? fmaf(v, c.x, w * c.y) : fmaf(v, c.x, -w * c.y);
+}
+
+// sigmoid of the output gate's pre-activation of (token, head); 1 without a gate
+template <typename T>
+__device__ __forceinline__ float out_gate(const LatentAttnArgs& a, long long t, int h) {
+  if (!a.gate) return 1.0f;
+  return 1.0f / (1.0f + expf(-ldf(static_cast<const T*>(a.gate) + t * a.ldg + h)));
+}
+
 // one CTA per token
 template <typename T>
 __global__ void __launch_bounds__(128) latent_prep_kernel(LatentPrepArgs a) {
   __shared__ float red[8];
   const int t = blockIdx.x;
   const int C = a.kv_rank, R = a.rot_dim, D = a.dim;
-  const T* d = static_cast<const T*>(a.dkv) + static_cast<long long>(t) * a.lddkv;
-  const int pos = a.positions[t];
-  T* row = static_cast<T*>(a.cache) + static_cast<long long>(a.slots[t]) * (C + R);
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < C; i += blockDim.x) { const float v = ldf(d + i); ss = fmaf(v, v, ss); }
-  ss = block_sum(ss, red);
-  const float inv = 1.0f / sqrtf(ss / static_cast<float>(C) + a.eps);
-  for (int i = threadIdx.x; i < C; i += blockDim.x) stf(row + i, ldf(d + i) * inv * a.norm_w[i]);
-  const int half = a.rot_dims / 2;
-  const float2* cs = a.rope + static_cast<long long>(pos) * half;
-  // shared rotated key part
-  for (int i = threadIdx.x; i < R; i += blockDim.x) {
-    const int pr = i >> 1;
-    float v = ldf(d + C + i);
-    if (pr < half) {
-      const float u0 = ldf(d + C + 2 * pr), u1 = ldf(d + C + 2 * pr + 1);
-      const float2 c = cs[pr];
-      v = (i & 1) ? fmaf(u1, c.x, u0 * c.y) : fmaf(u0, c.x, -u1 * c.y);
-    }
-    stf(row + C + i, v);
+  if (a.cq) {
+    const T* u = static_cast<const T*>(a.cq) + static_cast<long long>(t) * a.ldcq;
+    T* o = static_cast<T*>(a.cq_out) + static_cast<long long>(t) * a.ldcq_out;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) { const float v = ldf(u + i); ss = fmaf(v, v, ss); }
+    ss = block_sum(ss, red);
+    const float inv = 1.0f / sqrtf(ss / static_cast<float>(a.q_rank) + a.eps);
+    for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) stf(o + i, ldf(u + i) * inv * a.cq_w[i]);
   }
-  // rotated part of every query head -> tail of the latent query
-  const T* q = static_cast<const T*>(a.q) + static_cast<long long>(t) * a.ldq;
-  float* ql = a.qlat + static_cast<long long>(t) * a.heads * (C + R);
-  for (int e = threadIdx.x; e < a.heads * R; e += blockDim.x) {
-    const int h = e / R, i = e - h * R, pr = i >> 1;
-    const T* qr = q + h * (D + R) + D;
-    float v = ldf(qr + i);
-    if (pr < half) {
-      const float u0 = ldf(qr + 2 * pr), u1 = ldf(qr + 2 * pr + 1);
-      const float2 c = cs[pr];
-      v = (i & 1) ? fmaf(u1, c.x, u0 * c.y) : fmaf(u0, c.x, -u1 * c.y);
+  const int half = a.rot_dims / 2;
+  const float2* cs = a.rope + static_cast<long long>(a.positions[t]) * half;
+  if (a.dkv) {
+    const T* d = static_cast<const T*>(a.dkv) + static_cast<long long>(t) * a.lddkv;
+    T* row = static_cast<T*>(a.cache) + static_cast<long long>(a.slots[t]) * (C + R);
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < C; i += blockDim.x) { const float v = ldf(d + i); ss = fmaf(v, v, ss); }
+    ss = block_sum(ss, red);
+    const float inv = 1.0f / sqrtf(ss / static_cast<float>(C) + a.eps);
+    for (int i = threadIdx.x; i < C; i += blockDim.x) stf(row + i, ldf(d + i) * inv * a.norm_w[i]);
+    // shared rotated key part
+    for (int i = threadIdx.x; i < R; i += blockDim.x) stf(row + C + i, rotated(d + C, i, half, a.half_pairs, cs));
+  }
+  if (a.q) {
+    // rotated part of every query head -> tail of the latent query
+    const T* q = static_cast<const T*>(a.q) + static_cast<long long>(t) * a.ldq;
+    float* ql = a.qlat + static_cast<long long>(t) * a.heads * (C + R);
+    for (int e = threadIdx.x; e < a.heads * R; e += blockDim.x) {
+      const int h = e / R, i = e - h * R;
+      ql[h * (C + R) + C + i] = rotated(q + h * (D + R) + D, i, half, a.half_pairs, cs);
     }
-    ql[h * (C + R) + C + i] = v;
   }
 }
 
-// one CTA per (token, head); dynamic shared memory: qlat row [C + R] + scores [window]
+// One CTA per (token, head).  The visible keys are walked in rounds of kRoundKeys with a running maximum and sum (any number
+// of keys); dynamic shared memory: the query row [C + R], the latent sum [C], one round of scores.
+constexpr int kRoundKeys = 1024;
 template <typename T>
 __global__ void __launch_bounds__(128) latent_attn_kernel(LatentAttnArgs a) {
   extern __shared__ float sm[];
@@ -102,7 +122,8 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(LatentAttnArgs a) {
   const int t = blockIdx.x, h = blockIdx.y;
   const int C = a.kv_rank, E = a.kv_rank + a.rot_dim;
   float* qs = sm;
-  float* sc = sm + E;
+  float* acc = qs + E;      // [C], column i owned by thread i % blockDim.x
+  float* sc = acc + C;      // [kRoundKeys]
   const int p = a.positions[t];
   const int lo = max(0, p - a.window + 1);
   const int nk = p - lo + 1;
@@ -110,38 +131,45 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(LatentAttnArgs a) {
   const T* cache = static_cast<const T*>(a.cache);
   const float* ql = a.qlat + (static_cast<long long>(t) * a.heads + h) * E;
   for (int i = threadIdx.x; i < E; i += blockDim.x) qs[i] = ql[i];
-  __syncthreads();
+  for (int i = threadIdx.x; i < C; i += blockDim.x) acc[i] = 0.f;
   const int lane = threadIdx.x & 31, wrp = threadIdx.x >> 5, nw = blockDim.x >> 5;
-  float mx = -FLT_MAX;
-  for (int jj = wrp; jj < nk; jj += nw) {
+  float m = a.sink ? a.sink[h] : -FLT_MAX, l = a.sink ? 1.f : 0.f;
+  auto row_of = [&](int jj) {
     const int j = lo + jj;
-    const T* kr = cache + (static_cast<long long>(bt[j / a.page]) * a.page + j % a.page) * E;
-    float s = 0.f;
-    for (int i = lane; i < E; i += 32) s = fmaf(qs[i], ldf(kr + i), s);
-    for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
-    s *= a.scale;
-    if (lane == 0) sc[jj] = s;
-    mx = fmaxf(mx, s);
-  }
-  mx = block_max(mx, red);   // includes the barrier that publishes sc[]
-  float sum = 0.f;
-  for (int jj = threadIdx.x; jj < nk; jj += blockDim.x) {
-    const float e = expf(sc[jj] - mx);
-    sc[jj] = e;
-    sum += e;
-  }
-  sum = block_sum(sum, red);
-  const float inv = 1.0f / sum;
-  float* out = a.olat + (static_cast<long long>(t) * a.heads + h) * C;
-  for (int i = threadIdx.x; i < C; i += blockDim.x) {
-    float acc = 0.f;
-    for (int jj = 0; jj < nk; ++jj) {
-      const int j = lo + jj;
-      const T* kr = cache + (static_cast<long long>(bt[j / a.page]) * a.page + j % a.page) * E;
-      acc = fmaf(sc[jj], ldf(kr + i), acc);
+    return cache + (static_cast<long long>(bt[j / a.page]) * a.page + j % a.page) * E;
+  };
+  for (int k0 = 0; k0 < nk; k0 += kRoundKeys) {
+    const int kn = min(kRoundKeys, nk - k0);
+    __syncthreads();   // the query is staged; the last round's scores are no longer read
+    float mx = -FLT_MAX;
+    for (int jj = wrp; jj < kn; jj += nw) {
+      const T* kr = row_of(k0 + jj);
+      float s = 0.f;
+      for (int i = lane; i < E; i += 32) s = fmaf(qs[i], ldf(kr + i), s);
+      for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+      s *= a.scale;
+      if (lane == 0) sc[jj] = s;
+      mx = fmaxf(mx, s);
     }
-    out[i] = acc * inv;
+    const float m_new = fmaxf(m, block_max(mx, red));   // includes the barrier that publishes sc[]
+    const float al = m == -FLT_MAX ? 0.f : expf(m - m_new);
+    float sum = 0.f;
+    for (int jj = threadIdx.x; jj < kn; jj += blockDim.x) {
+      const float e = expf(sc[jj] - m_new);
+      sc[jj] = e;
+      sum += e;
+    }
+    l = fmaf(l, al, block_sum(sum, red));
+    m = m_new;
+    for (int i = threadIdx.x; i < C; i += blockDim.x) {
+      float v = acc[i] * al;
+      for (int jj = 0; jj < kn; ++jj) v = fmaf(sc[jj], ldf(row_of(k0 + jj) + i), v);
+      acc[i] = v;
+    }
   }
+  const float inv = out_gate<T>(a, t, h) / l;
+  float* out = a.olat + (static_cast<long long>(t) * a.heads + h) * C;
+  for (int i = threadIdx.x; i < C; i += blockDim.x) out[i] = acc[i] * inv;
 }
 
 // ---------------------------------------------------------------- tensor-core kernel (bf16 cache)
@@ -235,7 +263,13 @@ __global__ void __launch_bounds__(256) latent_attn_mma_kernel(LatentAttnArgs a, 
       *reinterpret_cast<__nv_bfloat162*>(Qs + r * LDE + c + 2) = __floats2bfloat162_rn(v.z, v.w);
     }
   }
-  if (tid < R) { Ms[tid] = -FLT_MAX; Ls[tid] = 0.f; As[tid] = 1.f; }
+  if (tid < R) {
+    const int h = h0 + tid % HB;
+    const bool sink = a.sink && h < a.heads && blockIdx.z == 0;
+    Ms[tid] = sink ? a.sink[h] : -FLT_MAX;
+    Ls[tid] = sink ? 1.f : 0.f;
+    As[tid] = 1.f;
+  }
   float acc[MB][kMaxPairs][2][4];
 #pragma unroll
   for (int mb = 0; mb < MB; ++mb)
@@ -369,12 +403,11 @@ __global__ void __launch_bounds__(256) latent_attn_mma_kernel(LatentAttnArgs a, 
       const int r = mb * 16 + g + 8 * half, tq = r / HB, h = h0 + r % HB;
       if (tq >= ntq || h >= a.heads) continue;
       const long long orow = static_cast<long long>(tok0 + tq0 + tq) * a.heads + h;
-      float inv = 1.0f / Ls[r];
+      float inv = nsplit > 1 ? 1.0f : out_gate<bf16>(a, tok0 + tq0 + tq, h) / Ls[r];
       float* out = a.olat + orow * C;
       if (nsplit > 1) {
         // partial: [row][split][C + 2] = unnormalised sums, running maximum, running sum
         out = split_ws + (orow * nsplit + blockIdx.z) * (C + 2);
-        inv = 1.0f;
         if (w == 0 && t4 == 0) { out[C] = Ms[r]; out[C + 1] = Ls[r]; }
       }
 #pragma unroll
@@ -391,7 +424,7 @@ __global__ void __launch_bounds__(256) latent_attn_mma_kernel(LatentAttnArgs a, 
 }
 
 // one warp per (token, head): combine the splits' partials
-__global__ void latent_attn_merge_kernel(const float* ws, float* olat, int C, int nsplit, long long rows) {
+__global__ void latent_attn_merge_kernel(LatentAttnArgs a, const float* ws, float* olat, int C, int nsplit, long long rows) {
   const long long row = static_cast<long long>(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (row >= rows) return;
   const int lane = threadIdx.x & 31;
@@ -403,7 +436,7 @@ __global__ void latent_attn_merge_kernel(const float* ws, float* olat, int C, in
     const float m = p[s * (C + 2) + C];
     if (m != -FLT_MAX) L += p[s * (C + 2) + C + 1] * expf(m - M);
   }
-  const float inv = 1.0f / L;
+  const float inv = out_gate<bf16>(a, row / a.heads, static_cast<int>(row % a.heads)) / L;
   for (int c = lane; c < C; c += 32) {
     float acc = 0.f;
     for (int s = 0; s < nsplit; ++s) {
@@ -487,7 +520,13 @@ __global__ void __launch_bounds__(256) latent_attn_mma_wide_kernel(LatentAttnArg
       *reinterpret_cast<__nv_bfloat162*>(Qs + r * LDE + c + 2) = __floats2bfloat162_rn(v.z, v.w);
     }
   }
-  if (tid < R) { Ms[tid] = -FLT_MAX; Ls[tid] = 0.f; As[tid] = 1.f; }
+  if (tid < R) {
+    const int h = h0 + tid % HB;
+    const bool sink = a.sink && h < a.heads;
+    Ms[tid] = sink ? a.sink[h] * 1.4426950408889634f : -FLT_MAX;   // in the unit of the scores below
+    Ls[tid] = sink ? 1.f : 0.f;
+    As[tid] = 1.f;
+  }
   float acc[MB][kMaxPairs][2][4];
 #pragma unroll
   for (int mb = 0; mb < MB; ++mb)
@@ -638,7 +677,7 @@ __global__ void __launch_bounds__(256) latent_attn_mma_wide_kernel(LatentAttnArg
     for (int half = 0; half < 2; ++half) {
       const int r = mb * 16 + g + 8 * half, tq = r / HB, h = h0 + r % HB;
       if (tq >= ntq || h >= a.heads) continue;
-      const float inv = 1.0f / Ls[r];
+      const float inv = out_gate<bf16>(a, tok0 + tq0 + tq, h) / Ls[r];
       float* out = a.olat + (static_cast<long long>(tok0 + tq0 + tq) * a.heads + h) * C;
 #pragma unroll
       for (int i = 0; i < kMaxPairs; ++i) {
@@ -682,6 +721,7 @@ int rope_table_interleaved(float2* table, int max_pos, int dims, double base, cu
 int latent_prep(const LatentPrepArgs& a, cudaStream_t st) {
   if (a.T <= 0) return 0;
   if (a.rot_dims > a.rot_dim || a.rot_dims % 2) return -1;
+  if (a.cq && (!a.cq_w || !a.cq_out || a.q_rank < 1)) return -1;
   if (a.t == DT_BF16) latent_prep_kernel<bf16><<<a.T, 128, 0, st>>>(a);
   else latent_prep_kernel<float><<<a.T, 128, 0, st>>>(a);
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
@@ -736,11 +776,11 @@ int latent_attention(const LatentAttnArgs& a, cudaStream_t st) {
     if (cudaGetLastError() != cudaSuccess) return -2;
     if (nsplit > 1) {
       const long long rows = static_cast<long long>(a.T) * a.heads;
-      latent_attn_merge_kernel<<<static_cast<unsigned>((rows + 3) / 4), 128, 0, st>>>(a.split_ws, a.olat, a.kv_rank, nsplit, rows);
+      latent_attn_merge_kernel<<<static_cast<unsigned>((rows + 3) / 4), 128, 0, st>>>(a, a.split_ws, a.olat, a.kv_rank, nsplit, rows);
     }
     return cudaGetLastError() == cudaSuccess ? 0 : -2;
   }
-  const size_t smem = static_cast<size_t>(a.kv_rank + a.rot_dim + a.window) * sizeof(float);
+  const size_t smem = static_cast<size_t>(2 * a.kv_rank + a.rot_dim + kRoundKeys) * sizeof(float);
   if (smem > 200 * 1024) return -1;
   dim3 grid(a.T, a.heads);
   if (a.t == DT_BF16) {

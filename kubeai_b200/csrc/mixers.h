@@ -23,7 +23,7 @@ enum DType { DT_BF16 = 0, DT_F32 = 1 };
 inline size_t dtype_bytes(DType t) { return t == DT_BF16 ? 2 : 4; }
 
 // ---------------------------------------------------------------- linear (linear.cu)
-enum LinearAct { LIN_NONE = 0, LIN_RELU2 = 1 };   // epilogue on the fp32 accumulator: identity, max(y, 0)^2
+enum LinearAct { LIN_NONE = 0, LIN_RELU2 = 1, LIN_XIELU = 2 };   // identity, max(y, 0)^2 (epilogues on the fp32 accumulator); xIELU (bias_act only)
 // Y[b][t, n] = act( sum_k X[b][row(t), k] * W[b'][n, k] ),  t < T, n < N.
 //   batch > 1: X, W, Y advance by xbs / wbs / ybs elements per batch index (per-head projections inside wider rows).
 //   x_rows (optional): row(t) = x_rows[t], a negative entry reads a zero row and its output row is not written.
@@ -79,7 +79,8 @@ int residual_dyt(float* x, const void* a, const void* f, DType ta, float mult, c
 int glu_clamped(const void* gu, int ldgu, void* y, int ldy, DType t, int T, int F, float limit, float slope, cudaStream_t st,
                 float up_offset = 1.0f);
 // y[t, i] = act(y[t, i] + bias[i]) in place, i < n (leading dimension ldy; bias fp32, may be null; act: LinearAct)
-int bias_act(void* y, int ldy, const float* bias, int act, DType t, int T, int n, cudaStream_t st);
+// LIN_XIELU: act(z) = a_pos z^2 + z / 2 for z > 0, a_neg (exp(z) - 1 - z) + z / 2 for z <= 0.
+int bias_act(void* y, int ldy, const float* bias, int act, DType t, int T, int n, cudaStream_t st, float a_pos = 0.f, float a_neg = 0.f);
 // y[t, i] *= sigmoid(g[t, i]), i < n (leading dimensions ldy, ldg)
 int sigmoid_gate(void* y, int ldy, const void* g, int ldg, DType t, int T, int n, cudaStream_t st);
 // p[i] = offset + scale * u_i, u uniform in [-1, 1) from a counter hash of (seed, i): seeded random weights for benchmarks
@@ -103,7 +104,15 @@ int argmax_f32(const float* logits, int* out, int S, int V, cudaStream_t st);
 // rope (optional, [position][rot_dims / 2] of (cos, sin)): the first rot_dims dimensions of every query and key head are
 // rotated by the token's position as they are read, dimension i paired with i + rot_dims / 2 (the rotate-half layout), in
 // fp32; k_scale multiplies the key after the rotation.
-enum GlaAct { GLA_ACT_NONE = 0, GLA_ACT_SILU = 1 };
+// fgate_lower (optional, fp32 [heads * dim]): the HGRN2 form.  The key columns hold forget-gate pre-activations g; with
+// s = sigmoid(g + z_bias) the channel decays by f = lower + (1 - lower) s and its key is 1 - f, S <- diag(f) S + (1 - f) v^T.
+// z is then unused.
+// dt_pre (optional, type t, [T, heads] with leading dimension ld_dt) with dt_bias and dt_rate (fp32 [heads]): the Mamba-2
+// form.  d = softplus(dt_pre + dt_bias); every channel of head h decays by exp(dt_rate[h] d) and the key is multiplied by d.
+// group: that many neighbouring heads share one query and key block (q and k are then heads / group x dim; v, the states
+// and the gates stay per head).
+// GLA_ACT_SILU_Q applies the SiLU to q only.
+enum GlaAct { GLA_ACT_NONE = 0, GLA_ACT_SILU = 1, GLA_ACT_SILU_Q = 2 };
 struct GlaArgs {
   const void* qkv; DType t; int ld, q_off, k_off, v_off;
   float* z; const float* z_bias; float inv_tau, q_scale;   // z is overwritten with the decays
@@ -116,6 +125,9 @@ struct GlaArgs {
   const float* tok_decay = nullptr; const float* tok_kscale = nullptr;
   float* nstate = nullptr; float* nq = nullptr;
   const float2* rope = nullptr; int rot_dims = 0; float k_scale = 1.f;
+  const float* fgate_lower = nullptr;
+  const void* dt_pre = nullptr; int ld_dt = 0; const float* dt_bias = nullptr; const float* dt_rate = nullptr;
+  int group = 1;
 };
 int gla_scan(const GlaArgs& a, cudaStream_t st);
 // y[t, h * vdim + :] (leading dimension ldy) = o[t, h, :] / sqrt(mean(o^2) + eps) * w * silu(g[t, h, :])   (w: fp32 [vdim], shared by the heads)
@@ -128,7 +140,7 @@ enum GateAct { GATE_SILU = 0, GATE_SIGMOID = 1 };
 // Per-head form only: w_full = true reads the weight as [heads * vdim] (every head its own) instead of [vdim]; with den_nq
 // and den_floor (fp32 [T, heads]) the outputs of head h are divided by max(|den_nq[t, h]|, den_floor[t, h]) + den_eps
 // before the norm (a normalised recurrence: den_nq is the product n . q of its running key sum with the query).
-// w may be null: a norm without a weight.
+// w may be null: a norm without a weight.  g may be null: no gate.
 struct OutGateArgs {
   const float* o; const void* g; int ldg; const float* w; float eps;
   void* y; int ldy; DType t;
@@ -138,6 +150,16 @@ struct OutGateArgs {
   const float* den_nq = nullptr; const float* den_floor = nullptr; float den_eps = 0.f;
 };
 int recurrent_out_gate(const OutGateArgs& a, cudaStream_t st);
+// The gate in front of the norm: u = (o[t, h, :] + skip[h] * x[t, h, :]) * silu(z[t, h, :]) over the concatenated heads; u is
+// cut into `groups` equal parts, every part divided by its own sqrt(mean(u^2) + eps), times w [heads * vdim].  skip may be
+// null (x is then unused).  o fp32 [T, heads * vdim]; x, z, y of type t; fp32 up to the rounding of y.
+struct GatedGroupNormArgs {
+  const float* o; const void* x; int ldx; const float* skip;
+  const void* z; int ldz; const float* w; float eps;
+  void* y; int ldy; DType t;
+  int T, heads, vdim, groups;
+};
+int gated_group_norm(const GatedGroupNormArgs& a, cudaStream_t st);
 // The scalar gates of the matrix-memory recurrence with exponential gating (mLSTM), per token and head, in fp32:
 //   log input gate  i = cap * tanh(zi / cap),   log forget gate  f = logsigmoid(cap * tanh(zf / cap))   (cap <= 0: no cap)
 //   running log-scale  m_t = max(f_t + m_(t-1), i_t),  m before the first token of a sequence is 0
@@ -159,6 +181,9 @@ int rope_table_interleaved(float2* table, int max_pos, int dims, double base, cu
 // the next rot_dim columns are rotated (first rot_dims of them) -> cache row tail; the rotated part of every query head
 // (q laid out [heads][dim + rot_dim]) is rotated into qlat[t][h][kv_rank ...] (fp32, row stride heads * (kv_rank + rot_dim)).
 // cache: [slot][kv_rank + rot_dim] of type t, slot = page * page_size + offset as given by slots[t].
+// Parts are optional: q null rotates no queries (they may need a projection that comes later), dkv null writes no cache row
+// (a layer that reads another layer's rows).  cq (optional): a query latent [T, q_rank] that is unit-RMS-normed (same eps)
+// and scaled by cq_w into cq_out.  half_pairs: rotation pairs are (i, i + rot_dims / 2) instead of (2i, 2i + 1).
 struct LatentPrepArgs {
   const void* q; int ldq; const void* dkv; int lddkv; DType t;
   const float* norm_w; float eps;
@@ -166,10 +191,15 @@ struct LatentPrepArgs {
   const int* positions; const int* slots;
   void* cache; float* qlat;
   int T, heads, dim, rot_dim, kv_rank;
+  bool half_pairs = false;
+  const void* cq = nullptr; int ldcq = 0; const float* cq_w = nullptr; int q_rank = 0; void* cq_out = nullptr; int ldcq_out = 0;
 };
 int latent_prep(const LatentPrepArgs& a, cudaStream_t st);
 // Sliding-window softmax attention in latent space: for token t at position p of sequence s, keys j with
 // max(0, p - window + 1) <= j <= p; score = qlat[t, h] . cache[j] * scale; olat[t, h] = sum_j softmax_j * cache[j][:kv_rank].
+// sink (optional, fp32 [heads]): the softmax denominator of head h gets the extra term exp(sink[h]), which belongs to no
+// cached token, adds nothing to the sum and stays outside scale.  gate (optional, type t, leading dimension ldg): olat[t, h]
+// is multiplied by sigmoid(gate[t * ldg + h]).
 struct LatentAttnArgs {
   const float* qlat; const void* cache; DType t;
   const int* positions; const int* seq_of_tok; const int* block_tables; int max_blocks, page;
@@ -178,6 +208,8 @@ struct LatentAttnArgs {
   const int* seqs; int nseq;   // the step's per-sequence table ({first row, rows, first position, ...}); needed by the tensor-core kernel
   int max_ctx;                 // longest context (position of a last token + 1) in the step, for the split decision
   float* split_ws; long long split_ws_floats;   // optional workspace of the split form: [rows][splits][kv_rank + 2] fp32
+  const float* sink = nullptr;
+  const void* gate = nullptr; int ldg = 0;
 };
 int latent_attention(const LatentAttnArgs& a, cudaStream_t st);
 
@@ -335,15 +367,17 @@ int embed_sinusoid(const void* embed, DType tw, const int* ids, const int* pos, 
                    cudaStream_t st);
 // One boundary between two sublayers of a design with a norm on both sides of every sublayer, on one fp32 residual.
 // For r < rows, t = row_index ? row_index[r] : r:
-//   if (y)  u = y[t] + y_bias;  x[t] <- x[t] + (post_w ? u / sqrt(mean(u^2) + eps) * post_w : u)      (y_bias fp32, may be null)
+//   if (y)  u = y[t] + y_bias;  x[t] <- x[t] + mult * (post_w ? u / sqrt(mean(u^2) + eps) * post_w : u)      (y_bias fp32, may be null)
 //   if (h)  h[r] = pre_w ? x[t] / sqrt(mean(x[t]^2) + eps) * pre_w : x[t]                             (fp32 statistics; h of type th)
-// post_w and pre_w are the multiplicative weights themselves (a stored offset from one is added at load).
+// post_w and pre_w are the multiplicative weights themselves (a stored offset from one is added at load).  Without post_w
+// this is the boundary of a pre-norm design with a residual multiplier.
 struct SandwichArgs {
   float* x;
   const void* y; DType ty; const float* y_bias;
   const float* post_w; const float* pre_w; float eps;
   void* h; DType th;
   const int* row_index; int rows; int W;
+  float mult = 1.f;
 };
 int sandwich_step(const SandwichArgs& a, cudaStream_t st);
 

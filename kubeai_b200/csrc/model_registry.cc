@@ -14,6 +14,7 @@ const Entry kModels[] = {
     {"Zinavik", make_zinavik},
     {"Mulenex", make_mulenex},
     {"Nagilix", make_nagilix},
+    {"Soselix", make_soselix},
 };
 }  // namespace
 

@@ -62,15 +62,51 @@ __global__ void glu_clamped_kernel(const T* gu, int ldgu, T* y, int ldy, int F, 
   stf(y + t * ldy + c, g * sigmoidf_(slope * g) * (u + up_offset));
 }
 
+__device__ __forceinline__ float act_of(float v, int act, float a_pos, float a_neg) {
+  if (act == LIN_RELU2) { v = fmaxf(v, 0.f); return v * v; }
+  if (act == LIN_XIELU) return fmaf(v > 0.f ? a_pos * v : 0.5f, v, v > 0.f ? 0.5f * v : a_neg * (expm1f(v) - v));
+  return v;
+}
+
 template <typename T>
-__global__ void bias_act_kernel(T* y, int ldy, const float* bias, int act, int n, long long total) {
+__global__ void bias_act_kernel(T* y, int ldy, const float* bias, int act, int n, long long total, float a_pos, float a_neg) {
   const long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x;
   if (i >= total) return;
   const long long t = i / n;
   const int c = static_cast<int>(i - t * n);
-  float v = ldf(y + t * ldy + c) + (bias ? bias[c] : 0.f);
-  if (act == LIN_RELU2) { v = fmaxf(v, 0.f); v = v * v; }
-  stf(y + t * ldy + c, v);
+  stf(y + t * ldy + c, act_of(ldf(y + t * ldy + c) + (bias ? bias[c] : 0.f), act, a_pos, a_neg));
+}
+
+// Rows of whole 16-byte pieces: a thread owns one piece of a column block and walks rows with its biases in registers.
+// grid: (column blocks of blockDim.x pieces, row blocks of `rows` rows)
+template <typename T>
+__global__ void __launch_bounds__(128) bias_act_vec_kernel(T* y, int ldy, const float* bias, int act, int n, int rows, int T_, float a_pos, float a_neg) {
+  constexpr int V = 16 / sizeof(T);
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V;
+  if (c >= n) return;
+  float b[V];
+#pragma unroll
+  for (int i = 0; i < V; ++i) b[i] = bias ? __ldg(bias + c + i) : 0.f;
+  const int t0 = blockIdx.y * rows, t1 = min(T_, t0 + rows);
+#pragma unroll 4
+  for (int t = t0; t < t1; ++t) {
+    uint4* p = reinterpret_cast<uint4*>(y + static_cast<long long>(t) * ldy + c);
+    const uint4 r = *p;
+    uint32_t u[4] = {r.x, r.y, r.z, r.w};
+    if constexpr (sizeof(T) == 2) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float lo = act_of(__uint_as_float(u[i] << 16) + b[2 * i], act, a_pos, a_neg);
+        const float hi = act_of(__uint_as_float(u[i] & 0xffff0000u) + b[2 * i + 1], act, a_pos, a_neg);
+        const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
+        u[i] = *reinterpret_cast<const uint32_t*>(&v);
+      }
+    } else {
+#pragma unroll
+      for (int i = 0; i < 4; ++i) u[i] = __float_as_uint(act_of(__uint_as_float(u[i]) + b[i], act, a_pos, a_neg));
+    }
+    *p = make_uint4(u[0], u[1], u[2], u[3]);
+  }
 }
 
 template <typename T>
@@ -166,12 +202,22 @@ int glu_clamped(const void* gu, int ldgu, void* y, int ldy, DType t, int T, int 
   return done();
 }
 
-int bias_act(void* y, int ldy, const float* bias, int act, DType t, int T, int n, cudaStream_t st) {
+int bias_act(void* y, int ldy, const float* bias, int act, DType t, int T, int n, cudaStream_t st, float a_pos, float a_neg) {
   const long long total = static_cast<long long>(T) * n;
   if (total <= 0) return 0;
+  const int V = 16 / static_cast<int>(dtype_bytes(t));
+  if (n % V == 0 && ldy % V == 0 && reinterpret_cast<uintptr_t>(y) % 16 == 0) {
+    const int cb = (n / V + 127) / 128;
+    int rows = 8;   // fewer where that leaves SMs without work
+    while (rows > 1 && static_cast<long long>(cb) * ((T + rows - 1) / rows) < 8 * 148) rows >>= 1;
+    dim3 grid(cb, (T + rows - 1) / rows);
+    if (t == DT_BF16) bias_act_vec_kernel<bf16><<<grid, 128, 0, st>>>(static_cast<bf16*>(y), ldy, bias, act, n, rows, T, a_pos, a_neg);
+    else bias_act_vec_kernel<float><<<grid, 128, 0, st>>>(static_cast<float*>(y), ldy, bias, act, n, rows, T, a_pos, a_neg);
+    return done();
+  }
   const unsigned grid = static_cast<unsigned>((total + 255) / 256);
-  if (t == DT_BF16) bias_act_kernel<bf16><<<grid, 256, 0, st>>>(static_cast<bf16*>(y), ldy, bias, act, n, total);
-  else bias_act_kernel<float><<<grid, 256, 0, st>>>(static_cast<float*>(y), ldy, bias, act, n, total);
+  if (t == DT_BF16) bias_act_kernel<bf16><<<grid, 256, 0, st>>>(static_cast<bf16*>(y), ldy, bias, act, n, total, a_pos, a_neg);
+  else bias_act_kernel<float><<<grid, 256, 0, st>>>(static_cast<float*>(y), ldy, bias, act, n, total, a_pos, a_neg);
   return done();
 }
 
