@@ -3,7 +3,8 @@ and feed-forward sizes, on random weights (`bench.py --design nomanex`: beside t
 `bench.py --design zinavik`: beside Nomanex, whose recurrent scan, windowed attention and routed experts are the like
 kernels; `bench.py --design mulenex`: beside Zinavik, which runs the same attention, scan, routing and projection kernels;
 `bench.py --design nagilix`: beside Zinavik, whose streams, paged attention, constant-decay scan and clamped routed experts
-are the like kernels).  Every number is CUDA-event time of the engine's
+are the like kernels; `bench.py --design soselix`: beside Nomanex with dense feed-forwards in every layer, whose latent
+attention, recurrent scan and projections are the like kernels).  Every number is CUDA-event time of the engine's
 own step (b200_feed_step: the same packing, page pool, state slots and kernels as a scheduled step), after warm-up
 steps, with a buffer larger than L2 written between timed steps.  Per-kernel times come from a separate pass in which
 each launch is bracketed by events (b200_engine_profile_kernels for the design, b200_engine_profile_range for Llama),
@@ -68,6 +69,24 @@ def nagilix_config(z):
     ma = dict(type="mamba1", mixer=dict(inner=2 * W, state=16, dt_rank=W // 16, conv=4), mlp=mo)
     return dict(architecture="Nagilix", vocab=z["vocab"], width=W, norm=dict(eps=1e-5), logit_scale=1.0, max_positions=4096, streams=2,
                 layers=[pa, ma, pa, ma])
+
+
+def soselix_config(z):
+    H, W = z["heads"], z["width"]
+    la = dict(heads=H, dim=DIM, rot_dim=ROT, vdim=VDIM, kv_rank=RANK, q_rank=W // 2, rot=dict(base=10000.0, dims=ROT), scale=(DIM + ROT) ** -0.5)
+    hg = dict(heads=H, dim=DIM, vdim=VDIM)
+    ma = dict(heads=2 * W // 64, vdim=64, state=128, groups=8, norm_groups=8, conv=4)
+    dn = dict(kind="dense", ff=z["ff"])
+    layers = [dict(type="latent_attention", mixer=la, mlp=dn), dict(type="hgrn2", mixer=hg, mlp=dn), dict(type="mamba2", mixer=ma, mlp=dn),
+              dict(type="latent_attention", mixer=dict(la, kv_from=0), mlp=dn)]
+    return dict(architecture="Soselix", vocab=z["vocab"], width=W, residual_mult=0.5, norm=dict(eps=1e-5), embedding=dict(scale=1.0), layers=layers)
+
+
+def nomanex_dense_config(z):
+    c = nomanex_config(z)
+    for ly in c["layers"]:
+        ly["mlp"] = c["layers"][0]["mlp"]
+    return c
 
 
 def flush_l2(torch, buf):
@@ -148,7 +167,39 @@ def run_design(cfgj, lim, z, batch, prompt, decode_steps, warmup, peaks, torch, 
                     "projections_decode_frac_of_hbm": 2.0 * W * (n_in + k_out) / (us(kd, "proj_in") + us(kd, "proj_out")) / (hbm * 1e9),
                     # residual update + norm: reads the fp32 residual and two bf16 sublayer outputs, writes the residual and a bf16 row
                     "residual_norm_prefill_frac_of_hbm": nl * T * W * (4 + 4 + 2 + 2 + 2) / us(kp, "residual_norm") / (hbm * 1e9),
-                    "moe_experts_prefill_frac_of_bf16_peak": 2.0 * 2 * T * z["top"] * 2 * W * z["eff"] / (us(kp, "moe_up") + us(kp, "moe_down")) / (tf * 1e12),
+                    "latent_head_products_prefill_frac_of_bf16_peak": 2.0 * 2 * T * H * RANK * (DIM + VDIM) / (us(kp, "latent_q_absorb") + us(kp, "latent_v_expand")) / (tf * 1e12),
+                    "gla_out_gate_prefill_frac_of_hbm": 2.0 * T * H * VDIM * (4 + 2 + 2) / us(kp, "gla_out_gate") / (hbm * 1e9),
+                    "glu_prefill_frac_of_hbm": sum(T * ly["mlp"]["ff"] * 6.0 for ly in cfgj["layers"] if ly["mlp"]["kind"] == "dense") / us(kp, "glu") / (hbm * 1e9),
+                }
+                if "moe_up" in kp:
+                    r["roofline"]["moe_experts_prefill_frac_of_bf16_peak"] = 2.0 * 2 * T * z["top"] * 2 * W * z["eff"] / (us(kp, "moe_up") + us(kp, "moe_down")) / (tf * 1e12)
+            elif cfgj["architecture"] == "Soselix":
+                E, ma = RANK + ROT, cfgj["layers"][2]["mixer"]
+                L, Hm, N, P, F = len(cfgj["layers"]), ma["heads"], ma["state"], ma["vdim"], z["ff"]
+                qr, conv_c = cfgj["layers"][0]["mixer"]["q_rank"], Hm * P + 2 * ma["groups"] * N
+                keys = sum(p + 1 for p in range(prompt)) * batch
+                dkeys = batch * (prompt + 1)
+                proj = W * (2 * qr + E + 2 * H) + 2 * qr * H * (DIM + ROT) + 2 * W * H * VDIM          # the two attention layers
+                proj += W * (2 * H * DIM + H * VDIM) + W * H * VDIM + W * (Hm * P + conv_c + Hm) + W * Hm * P
+                proj += L * 2 * W * F
+                pk = lambda k: sum(us(k, n) for n in ("proj_in", "proj_q", "proj_out", "ff_up", "ff_down"))
+                calls = 2 * L + 1
+                r["roofline"] = {
+                    "latent_attention_prefill_frac_of_bf16_peak": 2.0 * 2 * H * keys * (E + RANK) / us(kp, "latent_attention") / (tf * 1e12),
+                    "hgrn2_scan_prefill_tflops": 6.0 * T * H * DIM * VDIM / us(kp, "hgrn2_scan") / 1e12,
+                    "mamba2_scan_prefill_tflops": 6.0 * T * Hm * N * P / us(kp, "mamba2_scan") / 1e12,
+                    "projections_prefill_frac_of_bf16_peak": 2.0 * T * proj / pk(kp) / (tf * 1e12),
+                    "hgrn2_scan_decode_frac_of_hbm": 2.0 * batch * H * DIM * VDIM * 4 / us(kd, "hgrn2_scan") / (hbm * 1e9),
+                    "mamba2_scan_decode_frac_of_hbm": 2.0 * batch * Hm * N * P * 4 / us(kd, "mamba2_scan") / (hbm * 1e9),
+                    "latent_attention_decode_frac_of_hbm": 2.0 * dkeys * E * 2 / us(kd, "latent_attention") / (hbm * 1e9),
+                    "projections_decode_frac_of_hbm": 2.0 * proj / pk(kd) / (hbm * 1e9),
+                    "latent_head_products_prefill_frac_of_bf16_peak": 2.0 * 2 * T * H * RANK * (DIM + VDIM) / (us(kp, "latent_q_absorb") + us(kp, "latent_v_expand")) / (tf * 1e12),
+                    # boundary: reads and writes the fp32 residual, reads a bf16 sublayer output, writes a bf16 row
+                    "residual_norm_prefill_frac_of_hbm": calls * T * W * (8.0 + 2 + 2) / us(kp, "residual_norm") / (hbm * 1e9),
+                    "ff_act_prefill_frac_of_hbm": L * T * F * 4.0 / us(kp, "ff_act") / (hbm * 1e9),
+                    "short_conv_prefill_frac_of_hbm": T * conv_c * 4.0 / us(kp, "short_conv") / (hbm * 1e9),
+                    "mamba2_gate_norm_prefill_frac_of_hbm": T * Hm * P * (4 + 2 + 2 + 2.0) / us(kp, "mamba2_gate_norm") / (hbm * 1e9),
+                    "hgrn2_out_norm_prefill_frac_of_hbm": T * H * VDIM * (4 + 2.0) / us(kp, "hgrn2_out_norm") / (hbm * 1e9),
                 }
             elif cfgj["architecture"] == "Nagilix":
                 par = [ly for ly in cfgj["layers"] if ly["type"] == "parallel"]
@@ -254,6 +305,11 @@ def bench_size(design, name, z, batch, prompt, decode_steps, warmup, peaks):
     lim["num_kv_blocks"] = batch * ((lim["max_model_len"] + 15) // 16)
     res = {"size": dict(z, batch=batch, prompt=prompt)}
     T = batch * prompt
+    if design == "soselix":
+        res["soselix"] = run_design(soselix_config(z), lim, z, batch, prompt, decode_steps, warmup, peaks, torch, buf)
+        res["nomanex"] = run_design(nomanex_dense_config(z), lim, z, batch, prompt, decode_steps, warmup, peaks, torch, buf)
+        del buf
+        return res
     if design == "nagilix":
         res["nagilix"] = run_design(nagilix_config(z), lim, z, batch, prompt, decode_steps, warmup, peaks, torch, buf)
         res["zinavik"] = run_design(zinavik_config(z), lim, z, batch, prompt, decode_steps, warmup, peaks, torch, buf)
@@ -316,8 +372,8 @@ def _k_out(ly):
 
 
 def run(design, peaks, sizes=None, batch=8, prompt=512, decode_steps=8, warmup=3):
-    if design not in ("nomanex", "zinavik", "mulenex", "nagilix"):
-        raise SystemExit("unknown design %r (known: nomanex, zinavik, mulenex, nagilix)" % design)
+    if design not in ("nomanex", "zinavik", "mulenex", "nagilix", "soselix"):
+        raise SystemExit("unknown design %r (known: nomanex, zinavik, mulenex, nagilix, soselix)" % design)
     out = {"design": design, "dtype": "bf16", "data": "synthetic (seeded random weights and tokens)", "peaks": dict(hbm_gbs=peaks[0], bf16_tflops=peaks[1], source=peaks[2]),
            "timing": "CUDA events around the engine step, median of the timed steps, %d warm-up steps, 320 MB written between steps" % warmup,
            "sizes": {}}

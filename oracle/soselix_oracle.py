@@ -19,7 +19,7 @@ import numpy as np
 
 
 def sigmoid(z):
-    return 0.5 * (1.0 + np.tanh(0.5 * np.asarray(z, dtype=np.float64)))
+    return np.exp(-np.logaddexp(0.0, -np.asarray(z, dtype=np.float64)))      # no overflow, small values keep their digits
 
 
 def silu(z):

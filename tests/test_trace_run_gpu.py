@@ -11,6 +11,7 @@ import pytest
 
 import mulenex_util as mx
 import nagilix_util as nx
+import soselix_util as sx
 from zinavik_util import layer, left, make_config, moe, oracle_for, random_weights, rel_err, right, write_model_dir
 
 pytestmark = pytest.mark.gpu
@@ -66,8 +67,16 @@ def nagilix_model():
     return cfg, W, nx.oracle_for(cfg, W)
 
 
+def soselix_model():
+    layers = [sx.latent(heads=6, dim=8, rot_dim=16, vdim=12, kv_rank=32, q_rank=24, mlp=sx.dense(48)), sx.mamba2(heads=4, vdim=16, state=8, mlp=None, norm_groups=2, conv=5),
+              sx.hgrn2(heads=3, dim=12, vdim=20), sx.latent(heads=2, dim=16, rot_dim=16, vdim=8, kv_rank=32, q_rank=16, kv_from=0, mlp=None)]
+    cfg = sx.make_config(layers, width=40, vocab=70)
+    W = sx.random_weights(cfg, seed=97)
+    return cfg, W, sx.oracle_for(cfg, W)
+
+
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("model", [zinavik_model, mulenex_model, nagilix_model])
+@pytest.mark.parametrize("model", [zinavik_model, mulenex_model, nagilix_model, soselix_model])
 def test_replayed_schedule_gives_the_oracles_logits(tmp_path, dtype, model):
     cfg, W, o = model()
     d = write_model_dir(tmp_path / "m", cfg, W)
