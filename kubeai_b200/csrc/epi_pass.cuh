@@ -7,6 +7,7 @@
 #include <cuda_bf16.h>
 #include <stdint.h>
 
+#include "activations.cuh"
 #include "gemm3.h"
 #include "ptx.cuh"
 
@@ -14,7 +15,7 @@ namespace b200 {
 
 // destination of the pair kernel's fused epilogue on steps of more than 128 tokens (gemm2_tcgen05.cu, mode 2)
 struct Gemm2Epi {
-  int epi;                 // GEMM3_EPI_PLAIN / RESADD / SILU / ROPE_KV
+  int epi;                 // GEMM3_EPI_PLAIN / RESADD / SILU / ROPE_KV / BIAS_XIELU
   __nv_bfloat16* out;      // PLAIN out [T, N]; RESADD residual in/out [T, N]; SILU act [T, N/2]; ROPE_KV the fused qkv buffer
   int ldo;
   const int* positions;    // ROPE_KV
@@ -25,6 +26,8 @@ struct Gemm2Epi {
   int* flags;              // one int per (unit, CTA rank): stamped with `epoch` when that unit's partial tile is in the workspace
   int epoch;
   int hybrid;              // whole-tile waves first, stream-K over the remaining tiles (A/B knob B200_GEMM_HYBRID=0)
+  const float* bias;       // BIAS_XIELU: out = xielu(y + bias) (activations.cuh), bias fp32 [N]
+  float a_pos, a_neg;
   int wide;                // 64-token epilogue rounds (two tcgen05.ld in flight); 0 = 32-token rounds (A/B knob B200_GEMM_WIDE_EPI=0)
 };
 
@@ -54,6 +57,20 @@ __device__ __forceinline__ void pass(const Gemm2Epi& E, const __nv_bfloat16* ob,
     for (int i = 0; i < 4; ++i) {
       const int item = et + i * 128, j = item >> 4, vv = item & 15, t = t_base + j;
       if (t < T) *reinterpret_cast<uint4*>(E.out + static_cast<size_t>(t) * E.ldo + n0 + vv * 8) = *reinterpret_cast<const uint4*>(ob + j * kRows + vv * 8);
+    }
+  } else if (E.epi == GEMM3_EPI_BIAS_XIELU) {
+    const int vv = et & 15;       // the thread's column piece is the same in every round
+    float b[8];
+    *reinterpret_cast<float4*>(b) = __ldg(reinterpret_cast<const float4*>(E.bias + n0 + vv * 8));
+    *reinterpret_cast<float4*>(b + 4) = __ldg(reinterpret_cast<const float4*>(E.bias + n0 + vv * 8 + 4));
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int j = (et + i * 128) >> 4, t = t_base + j;
+      V8 x;
+      x.u = *reinterpret_cast<const uint4*>(ob + j * kRows + vv * 8);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x.h[e] = __float2bfloat16_rn(xielu_fast(__bfloat162float(x.h[e]) + b[e], E.a_pos, E.a_neg));
+      if (t < T) *reinterpret_cast<uint4*>(E.out + static_cast<size_t>(t) * E.ldo + n0 + vv * 8) = x.u;
     }
   } else if (E.epi == GEMM3_EPI_RESADD) {
 #pragma unroll

@@ -911,7 +911,8 @@ int gemm_run_deferred(const GemmPlan& p, const CUtensorMap& tm_x, int block_n, v
 int gemm2_run_fused(const GemmPlan& p, const CUtensorMap& tm_x, int block_n, int T, const Gemm2Epi& e, cudaStream_t st) {
   if (T <= 0) return 0;
   if (p.N % (2 * kSlab) != 0 || e.ldo % 8 != 0 || !e.flags || !e.out) return -5;
-  if (e.epi != GEMM3_EPI_PLAIN && e.epi != GEMM3_EPI_RESADD && e.epi != GEMM3_EPI_SILU && e.epi != GEMM3_EPI_ROPE_KV) return -6;
+  if (e.epi != GEMM3_EPI_PLAIN && e.epi != GEMM3_EPI_RESADD && e.epi != GEMM3_EPI_SILU && e.epi != GEMM3_EPI_ROPE_KV && e.epi != GEMM3_EPI_BIAS_XIELU) return -6;
+  if (e.epi == GEMM3_EPI_BIAS_XIELU && !e.bias) return -5;
   const int ntt = (T + block_n - 1) / block_n;
   // one parked piece per unit: [unit][rank][block_n tokens][128 rows] fp32
   if (static_cast<size_t>(units_for(p, ntt)) * 2 * block_n * kSlab * sizeof(float) > p.ws_bytes) return -9;

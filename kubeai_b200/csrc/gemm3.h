@@ -9,7 +9,7 @@
 namespace b200 {
 
 enum { GEMM3_PRO_NONE = 0, GEMM3_PRO_NORM = 1 };
-enum { GEMM3_EPI_PLAIN = 0, GEMM3_EPI_RESADD = 1, GEMM3_EPI_SILU = 2, GEMM3_EPI_ROPE_KV = 3, GEMM3_EPI_ARGMAX = 4 };
+enum { GEMM3_EPI_PLAIN = 0, GEMM3_EPI_RESADD = 1, GEMM3_EPI_SILU = 2, GEMM3_EPI_ROPE_KV = 3, GEMM3_EPI_ARGMAX = 4, GEMM3_EPI_BIAS_XIELU = 5 };   // BIAS_XIELU: pair kernel only
 
 struct Gemm3Params {
   CUtensorMap tm_w;   // weight [N, K] bf16, box 128 rows x 64 cols, 128B swizzle (GemmPlan::tm_w)

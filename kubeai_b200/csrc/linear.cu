@@ -5,11 +5,17 @@
 // fp32 models, fp32 outputs (router logits, decay pre-activations, latent queries), odd sizes, gathers.
 //
 // Kernels: a 64 x 64 x 32 shared-memory tile kernel (fp32 weights: FMA, k ascending; bf16 weights: mma.sync tensor-core
-// products; either way one output element is accumulated in an order that does not depend on what else is in the batch), and a one-warp-per-output-row kernel for steps of at most 8 rows (decode), which
-// streams each weight row once with 16-byte loads.
+// products; either way one output element is accumulated in an order that does not depend on what else is in the batch), and
+// two kernels for the few rows of a decode step: up to 16 rows of a bf16 matrix whose rows are whole 16-byte pieces go through
+// mma.sync with the weights as the 16-row operand (every weight byte is loaded once, straight into fragments), anything else of
+// up to 8 rows through one warp per output row.
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
+#include <stdlib.h>
 
+#include <algorithm>
+
+#include "activations.cuh"
 #include "mixers.h"
 
 namespace b200 {
@@ -35,8 +41,12 @@ __device__ __forceinline__ void ld8(const bf16* p, float* o) {
     o[2 * i + 1] = __uint_as_float(u[i] & 0xffff0000u);
   }
 }
-__device__ __forceinline__ float apply_act(float v, int act) {
-  if (act == LIN_RELU2) { v = fmaxf(v, 0.f); v = v * v; }
+// bias and activation of one output element (TY: the type it is rounded to)
+template <typename TY>
+__device__ __forceinline__ float finish(const LinearArgs& a, float v, int n) {
+  if (a.bias) v += a.bias[n];
+  if (a.act == LIN_RELU2) { v = fmaxf(v, 0.f); v = v * v; }
+  else if (a.act == LIN_XIELU) v = sizeof(TY) == 2 ? xielu_fast(v, a.a_pos, a.a_neg) : xielu(v, a.a_pos, a.a_neg);
   return v;
 }
 
@@ -104,7 +114,7 @@ __global__ void __launch_bounds__(256) linear_tile_kernel(LinearArgs a) {
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = col0 + tx * 4 + j;
-      if (n < a.N) st1(Y + static_cast<long long>(t) * a.ldy + n, apply_act((a.row_scale ? acc[i][j] * rs : acc[i][j]) + (a.bias ? a.bias[n] : 0.f), a.act));
+      if (n < a.N) st1(Y + static_cast<long long>(t) * a.ldy + n, finish<TY>(a, a.row_scale ? acc[i][j] * rs : acc[i][j], n));
     }
   }
 }
@@ -221,7 +231,7 @@ __global__ void __launch_bounds__(256) linear_tile_mma_kernel(LinearArgs a) {
 #pragma unroll
       for (int j = 0; j < 2; ++j) {
         const int n = col0 + 32 * wn + 8 * nb + 2 * t4 + j;
-        if (n < a.N) st1(Y + static_cast<long long>(t) * a.ldy + n, apply_act((a.row_scale ? acc[nb][2 * half + j] * rs : acc[nb][2 * half + j]) + (a.bias ? a.bias[n] : 0.f), a.act));
+        if (n < a.N) st1(Y + static_cast<long long>(t) * a.ldy + n, finish<TY>(a, a.row_scale ? acc[nb][2 * half + j] * rs : acc[nb][2 * half + j], n));
       }
   }
 }
@@ -259,8 +269,102 @@ __global__ void __launch_bounds__(256) linear_rows_kernel(LinearArgs a) {
       float v = acc[t];
 #pragma unroll
       for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-      if (lane == 0) st1(Y + static_cast<long long>(t) * a.ldy + n, apply_act((a.row_scale ? v * a.row_scale[t] : v) + (a.bias ? a.bias[n] : 0.f), a.act));
+      if (lane == 0) st1(Y + static_cast<long long>(t) * a.ldy + n, finish<TY>(a, a.row_scale ? v * a.row_scale[t] : v, n));
     }
+  }
+}
+
+// At most 8 * NB rows of X against a bf16 matrix: mma.sync m16n8k16 with 16 weight rows as the first operand and 8 tokens as
+// the second.  A lane loads 16 contiguous bytes (8 k) of its two weight rows and of its token's row; the k index inside a
+// 32-wide step is permuted the same way on both sides (lane piece t4 holds k 8 t4 .. 8 t4 + 7, its first half feeds the first
+// mma, its second half the second), so no fragment goes through shared memory.  The 8 warps of a CTA are KS slices of K times
+// 8 / KS groups of 16 weight rows; the slices' sums meet in shared memory and are added in a fixed order.  An fp32 X is split
+// into two bf16 terms, x = hi + lo up to 2^-16 of x.  The order of the sums depends on K alone.
+__device__ __forceinline__ uint4 ldx8(const bf16* p, uint4*) { return *reinterpret_cast<const uint4*>(p); }
+__device__ __forceinline__ uint4 ldx8(const float* p, uint4* lo) {
+  float v[8];
+  ld8(p, v);
+  uint32_t h[4], l[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const __nv_bfloat162 b = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+    const __nv_bfloat162 r = __floats2bfloat162_rn(v[2 * i] - __low2float(b), v[2 * i + 1] - __high2float(b));
+    h[i] = *reinterpret_cast<const uint32_t*>(&b);
+    l[i] = *reinterpret_cast<const uint32_t*>(&r);
+  }
+  *lo = make_uint4(l[0], l[1], l[2], l[3]);
+  return make_uint4(h[0], h[1], h[2], h[3]);
+}
+
+template <typename TX, typename TY, int NB, int U>
+__global__ void __launch_bounds__(256) linear_rows_mma_kernel(LinearArgs a, int KS) {
+  constexpr bool SPLIT = sizeof(TX) == 4;
+  __shared__ float part[8][16][8 * NB + 1];   // [warp][weight row][token]
+  const int lane = threadIdx.x & 31, wrp = threadIdx.x >> 5, g = lane >> 2, t4 = lane & 3;
+  const int ks = wrp % KS, RG = 8 / KS;
+  const int n0 = (blockIdx.x * RG + wrp / KS) * 16;
+  const long long b = blockIdx.z;
+  const bf16* W = static_cast<const bf16*>(a.W) + b * a.wbs;
+  const TX* X = static_cast<const TX*>(a.X) + b * a.xbs;
+  TY* Y = static_cast<TY*>(a.Y) + b * a.ybs;
+  const bool r0 = n0 + g < a.N, r1 = n0 + g + 8 < a.N;
+  const bf16* w0 = W + static_cast<long long>(n0 + g) * a.ldw;
+  const bf16* w1 = w0 + 8ll * a.ldw;
+  const TX* xr[NB];
+  bool xin[NB];
+#pragma unroll
+  for (int i = 0; i < NB; ++i) { xin[i] = g + 8 * i < a.T; xr[i] = X + static_cast<long long>(g + 8 * i) * a.ldx; }
+  float acc[NB][4];
+#pragma unroll
+  for (int i = 0; i < NB; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+  const int steps = (a.K + 31) >> 5, per = (steps + KS - 1) / KS, s1 = min(steps, (ks + 1) * per);
+  const uint4 zero = make_uint4(0, 0, 0, 0);
+  for (int s = ks * per; s < s1; s += U) {
+    uint4 wa[U], wb[U], xv[U][NB], xl[U][SPLIT ? NB : 1];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int k = (s + u) * 32 + t4 * 8;
+      const bool in = s + u < s1 && k < a.K;      // K is a multiple of 8: a piece is inside or outside as a whole
+      wa[u] = in && r0 ? __ldg(reinterpret_cast<const uint4*>(w0 + k)) : zero;
+      wb[u] = in && r1 ? __ldg(reinterpret_cast<const uint4*>(w1 + k)) : zero;
+#pragma unroll
+      for (int i = 0; i < NB; ++i) {
+        xv[u][i] = zero;
+        if (SPLIT) xl[u][i] = zero;
+        if (in && xin[i]) xv[u][i] = ldx8(xr[i] + k, &xl[u][SPLIT ? i : 0]);
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const uint32_t a0[4] = {wa[u].x, wb[u].x, wa[u].y, wb[u].y}, a1[4] = {wa[u].z, wb[u].z, wa[u].w, wb[u].w};
+#pragma unroll
+      for (int i = 0; i < NB; ++i) {
+        mma_16816(acc[i], a0, xv[u][i].x, xv[u][i].y);
+        mma_16816(acc[i], a1, xv[u][i].z, xv[u][i].w);
+        if (SPLIT) {
+          mma_16816(acc[i], a0, xl[u][i].x, xl[u][i].y);
+          mma_16816(acc[i], a1, xl[u][i].z, xl[u][i].w);
+        }
+      }
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < NB; ++i) {
+    part[wrp][g][8 * i + 2 * t4] = acc[i][0];
+    part[wrp][g][8 * i + 2 * t4 + 1] = acc[i][1];
+    part[wrp][g + 8][8 * i + 2 * t4] = acc[i][2];
+    part[wrp][g + 8][8 * i + 2 * t4 + 1] = acc[i][3];
+  }
+  __syncthreads();
+  for (int e = threadIdx.x; e < RG * 16 * 8 * NB; e += 256) {
+    const int r = e % (RG * 16), t = e / (RG * 16), rg = r >> 4;     // neighbouring threads: neighbouring output columns
+    const int n = blockIdx.x * RG * 16 + r;
+    if (t >= a.T || n >= a.N) continue;
+    float v = 0.f;
+    for (int k = 0; k < KS; ++k) v += part[rg * KS + k][r & 15][t];
+    st1(Y + static_cast<long long>(t) * a.ldy + n, finish<TY>(a, a.row_scale ? v * a.row_scale[t] : v, n));
   }
 }
 
@@ -286,7 +390,7 @@ __global__ void __launch_bounds__(256) linear_picked_rows_kernel(LinearArgs a, P
   }
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
-  if (lane == 0) st1(static_cast<TY*>(a.Y) + dst * a.ldy + n, apply_act((a.row_scale ? acc * a.row_scale[r] : acc) + (a.bias ? a.bias[n] : 0.f), a.act));
+  if (lane == 0) st1(static_cast<TY*>(a.Y) + dst * a.ldy + n, finish<TY>(a, a.row_scale ? acc * a.row_scale[r] : acc, n));
 }
 
 template <typename TX, typename TW, typename TY>
@@ -302,6 +406,21 @@ int launch_picked(const LinearArgs& a, const PickedRows& p, cudaStream_t st) {
 template <typename TX, typename TW, typename TY>
 int launch_linear(const LinearArgs& a, cudaStream_t st) {
   const bool few = a.T <= 8 && !a.x_rows && !a.tile_group;
+  if constexpr (sizeof(TW) == 2) {
+    // B200_LIN_MMA_ROWS: A/B knob, the most rows that take the fragment kernel (0: none)
+    static const int mma_rows = [] { const char* e = getenv("B200_LIN_MMA_ROWS"); return e ? std::min(16, std::max(0, atoi(e))) : 16; }();
+    const bool vec = a.K % 8 == 0 && a.ldx % 8 == 0 && a.ldw % 8 == 0 && a.xbs % 8 == 0 && a.wbs % 8 == 0 &&
+                     reinterpret_cast<uintptr_t>(a.X) % 16 == 0 && reinterpret_cast<uintptr_t>(a.W) % 16 == 0;
+    if (vec && a.T <= mma_rows && !a.x_rows && !a.tile_group) {
+      const int steps = (a.K + 31) / 32;
+      const int KS = steps >= 32 ? 8 : (steps >= 16 ? 4 : (steps >= 8 ? 2 : 1));
+      dim3 grid((a.N + 128 / KS - 1) / (128 / KS), 1, a.batch);
+      constexpr int U = sizeof(TX) == 4 ? 4 : 8;
+      if (a.T <= 8) linear_rows_mma_kernel<TX, TY, 1, U><<<grid, 256, 0, st>>>(a, KS);
+      else linear_rows_mma_kernel<TX, TY, 2, U / 2><<<grid, 256, 0, st>>>(a, KS);
+      return cudaGetLastError() == cudaSuccess ? 0 : -2;
+    }
+  }
   if (few) {
     const size_t ex = sizeof(TX), ew = sizeof(TW);
     const bool vec = a.K % 8 == 0 && a.ldx % 8 == 0 && a.ldw % 8 == 0 && a.xbs % 8 == 0 && a.wbs % 8 == 0 &&

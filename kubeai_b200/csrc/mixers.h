@@ -23,7 +23,9 @@ enum DType { DT_BF16 = 0, DT_F32 = 1 };
 inline size_t dtype_bytes(DType t) { return t == DT_BF16 ? 2 : 4; }
 
 // ---------------------------------------------------------------- linear (linear.cu)
-enum LinearAct { LIN_NONE = 0, LIN_RELU2 = 1, LIN_XIELU = 2 };   // identity, max(y, 0)^2 (epilogues on the fp32 accumulator); xIELU (bias_act only)
+// Epilogue on the fp32 accumulator: identity, max(y, 0)^2, or xIELU with its two coefficients,
+//   a_pos z^2 + z / 2 for z > 0,   a_neg (exp(z) - 1 - z) + z / 2 for z <= 0
+enum LinearAct { LIN_NONE = 0, LIN_RELU2 = 1, LIN_XIELU = 2 };
 // Y[b][t, n] = act( sum_k X[b][row(t), k] * W[b'][n, k] ),  t < T, n < N.
 //   batch > 1: X, W, Y advance by xbs / wbs / ybs elements per batch index (per-head projections inside wider rows).
 //   x_rows (optional): row(t) = x_rows[t], a negative entry reads a zero row and its output row is not written.
@@ -45,6 +47,7 @@ struct LinearArgs {
   int act;
   const float* row_scale;
   const float* bias;
+  float a_pos = 0.f, a_neg = 0.f;
 };
 inline LinearArgs linear_args(const void* X, DType tx, const void* W, DType tw, void* Y, DType ty, int T, int N, int K) {
   LinearArgs a = {X, W, Y, tx, tw, ty, T, N, K, K, K, N, 1, 0, 0, 0, nullptr, nullptr, LIN_NONE, nullptr, nullptr};
@@ -79,7 +82,6 @@ int residual_dyt(float* x, const void* a, const void* f, DType ta, float mult, c
 int glu_clamped(const void* gu, int ldgu, void* y, int ldy, DType t, int T, int F, float limit, float slope, cudaStream_t st,
                 float up_offset = 1.0f);
 // y[t, i] = act(y[t, i] + bias[i]) in place, i < n (leading dimension ldy; bias fp32, may be null; act: LinearAct)
-// LIN_XIELU: act(z) = a_pos z^2 + z / 2 for z > 0, a_neg (exp(z) - 1 - z) + z / 2 for z <= 0.
 int bias_act(void* y, int ldy, const float* bias, int act, DType t, int T, int n, cudaStream_t st, float a_pos = 0.f, float a_neg = 0.f);
 // y[t, i] *= sigmoid(g[t, i]), i < n (leading dimensions ldy, ldg)
 int sigmoid_gate(void* y, int ldy, const void* g, int ldg, DType t, int T, int n, cudaStream_t st);

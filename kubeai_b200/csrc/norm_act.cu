@@ -7,6 +7,7 @@
 #include <cuda_runtime.h>
 #include <float.h>
 
+#include "activations.cuh"
 #include "mixers.h"
 
 namespace b200 {
@@ -62,10 +63,12 @@ __global__ void glu_clamped_kernel(const T* gu, int ldgu, T* y, int ldy, int F, 
   stf(y + t * ldy + c, g * sigmoidf_(slope * g) * (u + up_offset));
 }
 
+// T: the type the result is rounded to
+template <typename T>
 __device__ __forceinline__ float act_of(float v, int act, float a_pos, float a_neg) {
   if (act == LIN_RELU2) { v = fmaxf(v, 0.f); return v * v; }
-  if (act == LIN_XIELU) return fmaf(v > 0.f ? a_pos * v : 0.5f, v, v > 0.f ? 0.5f * v : a_neg * (expm1f(v) - v));
-  return v;
+  if (act != LIN_XIELU) return v;
+  return sizeof(T) == 2 ? xielu_fast(v, a_pos, a_neg) : xielu(v, a_pos, a_neg);
 }
 
 template <typename T>
@@ -74,7 +77,7 @@ __global__ void bias_act_kernel(T* y, int ldy, const float* bias, int act, int n
   if (i >= total) return;
   const long long t = i / n;
   const int c = static_cast<int>(i - t * n);
-  stf(y + t * ldy + c, act_of(ldf(y + t * ldy + c) + (bias ? bias[c] : 0.f), act, a_pos, a_neg));
+  stf(y + t * ldy + c, act_of<T>(ldf(y + t * ldy + c) + (bias ? bias[c] : 0.f), act, a_pos, a_neg));
 }
 
 // Rows of whole 16-byte pieces: a thread owns one piece of a column block and walks rows with its biases in registers.
@@ -96,14 +99,14 @@ __global__ void __launch_bounds__(128) bias_act_vec_kernel(T* y, int ldy, const 
     if constexpr (sizeof(T) == 2) {
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
-        const float lo = act_of(__uint_as_float(u[i] << 16) + b[2 * i], act, a_pos, a_neg);
-        const float hi = act_of(__uint_as_float(u[i] & 0xffff0000u) + b[2 * i + 1], act, a_pos, a_neg);
+        const float lo = act_of<T>(__uint_as_float(u[i] << 16) + b[2 * i], act, a_pos, a_neg);
+        const float hi = act_of<T>(__uint_as_float(u[i] & 0xffff0000u) + b[2 * i + 1], act, a_pos, a_neg);
         const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
         u[i] = *reinterpret_cast<const uint32_t*>(&v);
       }
     } else {
 #pragma unroll
-      for (int i = 0; i < 4; ++i) u[i] = __float_as_uint(act_of(__uint_as_float(u[i]) + b[i], act, a_pos, a_neg));
+      for (int i = 0; i < 4; ++i) u[i] = __float_as_uint(act_of<T>(__uint_as_float(u[i]) + b[i], act, a_pos, a_neg));
     }
     *p = make_uint4(u[0], u[1], u[2], u[3]);
   }

@@ -30,6 +30,7 @@
 
 #include <algorithm>
 
+#include "epi_pass.cuh"
 #include "errors.h"
 #include "gemm.h"
 #include "model.h"
@@ -108,6 +109,10 @@ class Soselix : public Model {
   std::vector<void*> allocs;
   float* gemm_ws = nullptr;
   int* gemm_counters = nullptr;
+  int* gemm_flags = nullptr;     // of the fused form: two per CTA pair, stamped with the launch's number
+  int gemm_epoch = 0;
+  bool fuse = true;
+  int few_rows = 16;
   CUtensorMap xm_h[kGemmNumBlockN];
   bool use_tc = false;
 
@@ -239,6 +244,9 @@ class Soselix : public Model {
       s.rec_floats = static_cast<size_t>(HD) * s.vdim;
     }
     s.n_in = at;
+    // a wide row is filled up to whole 256-row weight tiles (rows of zeros nobody reads), which the fused GEMM form asks for
+    const int full = (at + 255) / 256 * 256;
+    if (at >= 1024 && full - at <= at / 8) s.n_in = full;
   }
 
   int inspect(const CheckpointReader& ck, std::string* err) override {
@@ -352,7 +360,9 @@ class Soselix : public Model {
     const size_t ws_bytes = std::max(gemm_workspace_bytes(env.sms), gemm_deferred_ws_bytes(env.sms));
     if (dalloc(&gemm_ws, ws_bytes)) return -3;
     const size_t n_counters = 2ull * (maxN / 128 + 2) * (env.Tcap / 32 + 2);
-    if (dalloc(&gemm_counters, n_counters * sizeof(int))) return -3;
+    if (dalloc(&gemm_counters, n_counters * sizeof(int)) || dalloc(&gemm_flags, static_cast<size_t>(env.sms) * 2 * sizeof(int))) return -3;
+    if (const char* e = getenv("B200_SX_FUSE")) fuse = atoi(e) != 0;              // A/B knobs
+    if (const char* e = getenv("B200_SX_FEW_ROWS")) few_rows = atoi(e);
     const int bns[kGemmNumBlockN] = {32, 64, 128, 256, 512};
     auto maps = [&](CUtensorMap* m, const void* X, int K) {
       for (int i = 0; i < kGemmNumBlockN; ++i)
@@ -528,12 +538,40 @@ class Soselix : public Model {
   }
 
   // ------------------------------------------------------------ forward
-  int project(const GemmPlan& plan, bool tc, const CUtensorMap* xm, const void* X, const void* Wm, void* Y, int T, int N, int K) {
-    if (tc) {
-      const int bn = gemm_block_n_for(T);
-      return gemm_run(plan, xm[gemm_block_n_index(bn)], bn, Y, N, T, env.stream);
+  // Y = X W^T, with bias and xIELU behind it where the epilogue is given.  Steps of up to 16 tokens stream the weights through
+  // linear.cu's fragment kernel.  Larger steps take the pair GEMM; in its fused form (whole 256-row tiles, at least one tile
+  // per CTA pair) every tile leaves through the epilogue, otherwise the epilogue is a pass of its own over the result.
+  struct Epilogue {
+    const float* bias = nullptr;
+    float a_pos = 0.f, a_neg = 0.f;
+  };
+  int project(const GemmPlan& plan, bool tc, const CUtensorMap* xm, const void* X, const void* Wm, void* Y, int T, int N, int K, const Epilogue* ep = nullptr) {
+    if (tc && T > few_rows) {
+      const int bn = block_n(plan, T);
+      if (fuse && N % 256 == 0 && T > 128 && N / 256 * ((T + bn - 1) / bn) >= plan.max_ctas / 2) {
+        Gemm2Epi e;
+        memset(&e, 0, sizeof(e));
+        e.epi = ep ? GEMM3_EPI_BIAS_XIELU : GEMM3_EPI_PLAIN;
+        e.out = static_cast<bf16*>(Y); e.ldo = N;
+        e.flags = gemm_flags; e.epoch = ++gemm_epoch;
+        if (ep) { e.bias = ep->bias; e.a_pos = ep->a_pos; e.a_neg = ep->a_neg; }
+        return gemm2_run_fused(plan, xm[gemm_block_n_index(bn)], bn, T, e, env.stream);
+      }
+      const int rc = gemm_run(plan, xm[gemm_block_n_index(bn)], bn, Y, N, T, env.stream);
+      return rc || !ep ? rc : bias_act(Y, N, ep->bias, LIN_XIELU, dt, T, N, env.stream, ep->a_pos, ep->a_neg);
     }
-    return linear(linear_args(X, dt, Wm, dt, Y, dt, T, N, K), env.stream);
+    LinearArgs la = linear_args(X, dt, Wm, dt, Y, dt, T, N, K);
+    if (ep) { la.bias = ep->bias; la.act = LIN_XIELU; la.a_pos = ep->a_pos; la.a_neg = ep->a_neg; }
+    return linear(la, env.stream);
+  }
+  // Token-tile size: where 512-token tiles neither fill the pairs nor are close enough to one whole tile per pair (that form
+  // takes up to 64 k-blocks), 256-token tiles give the fused form its tile per pair.
+  int block_n(const GemmPlan& p, int T) const {
+    const int bn = gemm_block_n_for(T), pairs = p.max_ctas / 2;
+    if (bn != 512 || !fuse || p.N % 256) return bn;
+    const int t512 = p.N / 256 * ((T + 511) / 512), t256 = p.N / 256 * ((T + 255) / 256);
+    const bool whole = p.K <= 4096 && t512 * 5 >= pairs * 3;
+    return t512 < pairs && !whole && t256 >= pairs ? 256 : bn;
   }
 
   // per-kernel device time (b200_engine_kernel_times): with profiling on, every launch is bracketed by events and waited for
@@ -672,8 +710,9 @@ class Soselix : public Model {
       pend.y = ao; pend.bias = nullptr;
       if (s.mlp) {
         KRN("residual_norm", sandwich_step(boundary(pend, w.norm2, h, nullptr, T), st));
-        KRN("ff_up", project(w.p_up, w.tc_up, xm_h, h, w.w_up, hid, T, s.ff, W));
-        KRN("ff_act", bias_act(hid, s.ff, w.up_b, LIN_XIELU, dt, T, s.ff, st, w.act_pos, w.act_neg));
+        Epilogue ep;
+        ep.bias = w.up_b; ep.a_pos = w.act_pos; ep.a_neg = w.act_neg;
+        KRN("ff_up", project(w.p_up, w.tc_up, xm_h, h, w.w_up, hid, T, s.ff, W, &ep));
         KRN("ff_down", project(w.p_down, w.tc_down, w.xm_hid, hid, w.w_down, fo, T, W, s.ff));
         pend.y = fo; pend.bias = w.down_b;
       }
