@@ -28,6 +28,7 @@ SOURCES = [
     "linear.cu",
     "norm_act.cu",
     "gla.cu",
+    "scan_chunk.cu",
     "latent_attention.cu",
     "moe.cu",
     "hyper.cu",

@@ -469,6 +469,16 @@ int gla_scan(const GlaArgs& a, cudaStream_t st) {
   if (a.nseq <= 0) return 0;
   if (a.dim < 1 || a.vdim < 1 || a.heads < 1) return -1;
   if (a.rope && (a.rot_dims < 2 || a.rot_dims % 2 || a.rot_dims > a.dim || a.act != GLA_ACT_NONE)) return -1;
+  if (a.group < 1 || a.heads % a.group || (a.group > 1 && !a.tok_decay && !a.dt_pre && !a.head_decay)) return -1;
+  if (a.dt_pre && (!a.dt_bias || !a.dt_rate || a.tok_decay || a.head_decay || a.fgate_lower || a.nstate)) return -1;
+  if (a.fgate_lower && (!a.z_bias || a.tok_decay || a.head_decay || a.rope || a.act == GLA_ACT_SILU)) return -1;
+  if (scan_chunk_fits(a)) {
+    // steps that bring portions: a chunk of 64 costs about as much as a few tokens one by one (B200_SCAN_CHUNK: A/B knob, the
+    // mean portion from which the chunked form runs; 0 = never)
+    const char* e = getenv("B200_SCAN_CHUNK");
+    const int from = e ? atoi(e) : 8;
+    if (from > 0 && a.T >= static_cast<long long>(from) * a.nseq) return scan_chunk(a, st);
+  }
   int P = 1;
   while (P * kRows < a.dim) P <<= 1;
   if (P > 32) return -1;   // dim <= 1024
@@ -490,9 +500,6 @@ int gla_scan(const GlaArgs& a, cudaStream_t st) {
   if (smem > 48 * 1024) return -1;
   if ((a.nstate != nullptr) != (a.nq != nullptr) || (a.nstate && !a.tok_decay)) return -1;
   if (a.nstate && rows_per_part > kNormRows * tcols) return -1;
-  if (a.group < 1 || a.heads % a.group || (a.group > 1 && !a.tok_decay && !a.dt_pre && !a.head_decay)) return -1;
-  if (a.dt_pre && (!a.dt_bias || !a.dt_rate || a.tok_decay || a.head_decay || a.fgate_lower || a.nstate)) return -1;
-  if (a.fgate_lower && (!a.z_bias || a.tok_decay || a.head_decay || a.rope || a.act == GLA_ACT_SILU)) return -1;
   if (a.tok_decay) {
     if (!a.tok_kscale || a.head_decay) return -1;
   } else if (!a.head_decay && !a.dt_pre && !a.fgate_lower) {

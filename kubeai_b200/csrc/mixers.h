@@ -132,6 +132,10 @@ struct GlaArgs {
   int group = 1;
 };
 int gla_scan(const GlaArgs& a, cudaStream_t st);
+// The chunked tensor-core form of the dt_pre scan (scan_chunk.cu; same result up to fp32 rounding), for the shapes it takes;
+// gla_scan chooses it for bf16 steps of prompt portions.
+bool scan_chunk_fits(const GlaArgs& a);
+int scan_chunk(const GlaArgs& a, cudaStream_t st);
 // y[t, h * vdim + :] (leading dimension ldy) = o[t, h, :] / sqrt(mean(o^2) + eps) * w * silu(g[t, h, :])   (w: fp32 [vdim], shared by the heads)
 int gla_out_gate(const float* o, const void* g, int ldg, const float* w, float eps, void* y, int ldy, DType t, int T, int heads, int vdim,
                  cudaStream_t st);

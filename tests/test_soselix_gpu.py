@@ -227,6 +227,43 @@ def test_bfloat16_large_prompt_step_takes_the_64_row_attention_kernel_by_itself(
     assert np.median(rel_err(got, plain.astype(np.float64))) < 0.02 and rel_err(got, plain.astype(np.float64)).max() < 0.1
 
 
+@pytest.mark.parametrize("heads,vdim,state,groups,norm_groups", [(4, 16, 16, 2, 2), (3, 64, 128, 1, 1), (6, 24, 48, 3, 2), (2, 136, 64, 1, 4), (8, 8, 112, 2, 1), (5, 72, 32, 5, 5)])
+def test_chunked_tensor_core_scan_equals_the_token_by_token_scan(tmp_path, monkeypatch, heads, vdim, state, groups, norm_groups):
+    """State and value sizes that the chunked form of the Mamba-2 recurrence takes (whole and partial blocks of state rows and
+    value columns, several chunks of 64, portions that end inside a chunk): it keeps fp32 precision, so only the rounding of
+    the layer's bf16 output can differ from the sequential scan."""
+    cfg, W, d = build(tmp_path, [mamba2(heads=heads, vdim=vdim, state=state, groups=groups, norm_groups=norm_groups, conv=4, mlp=None)], seed=5, width=64, vocab=60)
+    t = toks(333, 60, 6)
+    want = oracle_for(cfg, W).forward(t)
+    out = {}
+    for knob in ("1", "0"):          # from one token per portion; never
+        monkeypatch.setenv("B200_SCAN_CHUNK", knob)
+        with open_engine(d, dtype="bfloat16") as e:
+            out[knob] = (feed_whole(e, t), feed_portions(e, t, [100, 64, 1, 17, 2, 90, 1]))
+    for a, b in zip(out["1"], out["0"]):
+        close16(a, want)
+        r = rel_err(a, b.astype(np.float64))
+        assert np.median(r) < 1e-3 and r.max() < 0.01, (np.median(r), r.max())
+
+
+@pytest.mark.parametrize("rate,step", [(3.0, 6.0), (-7.0, -2.0), (0.0, -60.0)])
+def test_chunked_scan_at_extreme_decays(tmp_path, monkeypatch, rate, step):
+    """Decays that leave nothing of a state after one token (no factor may overflow), decays next to one, and step sizes of
+    zero."""
+    cfg, W, d = build(tmp_path, [mamba2(heads=4, vdim=16, state=32, groups=2, norm_groups=2, mlp=None)], seed=7, width=48, vocab=60,
+                      edit=lambda W: (W["l0.mix.A_log"].fill(rate), W["l0.mix.dt_bias"].fill(step)))
+    t = toks(200, 60, 8)
+    want = oracle_for(cfg, W).forward(t)
+    with open_engine(d, dtype="bfloat16") as e:
+        got = feed_whole(e, t)
+    monkeypatch.setenv("B200_SCAN_CHUNK", "0")
+    with open_engine(d, dtype="bfloat16") as e:
+        one = feed_whole(e, t)
+    assert np.isfinite(got).all()
+    close16(got, want)
+    assert rel_err(got, one.astype(np.float64)).max() < 0.02
+
+
 # ---------------------------------------------------------------- cutting a sequence
 def test_prefill_equals_token_by_token_decoding(mix):
     cfg, W, d, o = mix
