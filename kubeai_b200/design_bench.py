@@ -196,7 +196,6 @@ def run_design(cfgj, lim, z, batch, prompt, decode_steps, warmup, peaks, torch, 
                     "latent_head_products_prefill_frac_of_bf16_peak": 2.0 * 2 * T * H * RANK * (DIM + VDIM) / (us(kp, "latent_q_absorb") + us(kp, "latent_v_expand")) / (tf * 1e12),
                     # boundary: reads and writes the fp32 residual, reads a bf16 sublayer output, writes a bf16 row
                     "residual_norm_prefill_frac_of_hbm": calls * T * W * (8.0 + 2 + 2) / us(kp, "residual_norm") / (hbm * 1e9),
-                    "ff_act_prefill_frac_of_hbm": L * T * F * 4.0 / us(kp, "ff_act") / (hbm * 1e9),
                     "short_conv_prefill_frac_of_hbm": T * conv_c * 4.0 / us(kp, "short_conv") / (hbm * 1e9),
                     "mamba2_gate_norm_prefill_frac_of_hbm": T * Hm * P * (4 + 2 + 2 + 2.0) / us(kp, "mamba2_gate_norm") / (hbm * 1e9),
                     "hgrn2_out_norm_prefill_frac_of_hbm": T * H * VDIM * (4 + 2.0) / us(kp, "hgrn2_out_norm") / (hbm * 1e9),
