@@ -227,6 +227,25 @@ def test_bfloat16_large_prompt_step_takes_the_64_row_attention_kernel_by_itself(
     assert np.median(rel_err(got, plain.astype(np.float64))) < 0.02 and rel_err(got, plain.astype(np.float64)).max() < 0.1
 
 
+def test_fused_large_step_products_equal_the_plain_ones(tmp_path, monkeypatch):
+    """Matrices of whole 256-row tiles in a step with a tile per CTA pair and more take the fused GEMM form: bias and xIELU in
+    the epilogue of a wide up-projection, 256-token tiles for a deep down-projection, the filled-up input projection.  The
+    step's last token tiles are partial.  Rows of the first tokens are the oracle's; all rows are those of the plain form."""
+    layers = [hgrn2(heads=4, dim=96, vdim=104, mlp=dense(4352)), mamba2(heads=8, vdim=120, state=16, groups=1, norm_groups=4, conv=4, mlp=None)]
+    cfg, W, d = build(tmp_path, layers, seed=81, width=2048, vocab=64)
+    T = 4700
+    t = toks(T, 64, 82)
+    rows = sorted(set(range(24)) | set(range(100, T, 97)) | {255, 256, 511, 512, 4095, 4096, 4607, 4608, T - 1})
+    out = {}
+    for knob in ("1", "0"):
+        monkeypatch.setenv("B200_SX_FUSE", knob)
+        with open_engine(d, dtype="bfloat16", max_tokens=4704, max_seqs=1) as e:
+            out[knob] = feed_whole(e, t, rows)
+    close16(out["1"][:24], oracle_for(cfg, W).forward(t[:24]))
+    r = rel_err(out["1"], out["0"].astype(np.float64))
+    assert np.median(r) < 0.01 and r.max() < 0.05, (np.median(r), r.max())
+
+
 @pytest.mark.parametrize("heads,vdim,state,groups,norm_groups", [(4, 16, 16, 2, 2), (3, 64, 128, 1, 1), (6, 24, 48, 3, 2), (2, 136, 64, 1, 4), (8, 8, 112, 2, 1), (5, 72, 32, 5, 5)])
 def test_chunked_tensor_core_scan_equals_the_token_by_token_scan(tmp_path, monkeypatch, heads, vdim, state, groups, norm_groups):
     """State and value sizes that the chunked form of the Mamba-2 recurrence takes (whole and partial blocks of state rows and
