@@ -29,6 +29,7 @@ SOURCES = [
     "norm_act.cu",
     "gla.cu",
     "scan_chunk.cu",
+    "delta.cu",
     "latent_attention.cu",
     "moe.cu",
     "hyper.cu",
@@ -39,6 +40,7 @@ SOURCES = [
     "mulenex.cu",
     "nagilix.cu",
     "soselix.cu",
+    "dabodra.cu",
     "model_registry.cc",
     "abi_ops.cu",
     "engine.cu",

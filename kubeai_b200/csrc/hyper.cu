@@ -11,6 +11,7 @@
 // A gated write-back multiplies y by sigmoid(gate + bias), the gate being a projection of the sublayer's own input.
 // `embed_learned_pos` fills the streams with the token's embedding row plus a learned position row; `branch_norm_sum` is
 // the meeting point of two mixers that ran side by side, each RMS-normed over the width with its own weight.
+// `embed_normed` starts a residual from RMS-normed embedding rows.
 //
 // Beside it, for designs with one residual and a norm on BOTH sides of every sublayer (mixers.h SandwichArgs): the
 // sublayer's output is RMS-normed before it is added, x <- x + norm_post(y + bias), and the next sublayer reads
@@ -372,7 +373,35 @@ __global__ void __launch_bounds__(256) sandwich_step_kernel(SandwichArgs a) {
   }
 }
 
+// Embedding rows RMS-normed into the residual, and the rounded row the first sublayer reads: one CTA per token.
+template <typename TW, typename TH>
+__global__ void __launch_bounds__(256) embed_normed_kernel(const TW* embed, const int* ids, const float* w, float eps, float* x, TH* h, int W, int vocab) {
+  __shared__ float red[8];
+  const long long t = blockIdx.x;
+  const int id = ids[t] < 0 || ids[t] >= vocab ? 0 : ids[t];
+  const TW* e = embed + static_cast<long long>(id) * W;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < W; i += blockDim.x) { const float v = ldf(e + i); ss = fmaf(v, v, ss); }
+  const float inv = 1.0f / sqrtf(cta_sum(ss, red) / static_cast<float>(W) + eps);
+  for (int i = threadIdx.x; i < W; i += blockDim.x) {
+    const float v = ldf(e + i) * inv * w[i];
+    x[t * W + i] = v;
+    if (h) stf(h + t * W + i, v);
+  }
+}
+
 }  // namespace
+
+int embed_normed(const void* embed, DType tw, const int* ids, const float* w, float eps, float* x, void* h, DType th, int T, int W, int vocab,
+                 cudaStream_t st) {
+  if (T <= 0) return 0;
+  if (!embed || !ids || !w || !x || W < 1) return -1;
+#define EN(TW, TH) embed_normed_kernel<TW, TH><<<T, threads_for(W), 0, st>>>(static_cast<const TW*>(embed), ids, w, eps, x, static_cast<TH*>(h), W, vocab)
+  if (tw == DT_BF16) { if (th == DT_BF16) EN(bf16, bf16); else EN(bf16, float); }
+  else { if (th == DT_BF16) EN(float, bf16); else EN(float, float); }
+#undef EN
+  return cudaGetLastError() == cudaSuccess ? 0 : -2;
+}
 
 int sinusoid_freq_table(float2* freq, int W, double base, cudaStream_t st) {
   const int pairs = (W + 1) / 2;

@@ -180,6 +180,25 @@ struct MlstmGateArgs {
 };
 int mlstm_gates(const MlstmGateArgs& a, cudaStream_t st);
 
+// ---------------------------------------------------------------- gated delta rule (delta.cu)
+// Per sequence and head, in fp32: with k^ = k / sqrt(sum(k^2) + unit_eps), q^ = q_scale q / sqrt(sum(q^2) + unit_eps),
+//   beta = sigmoid(beta_pre),  g = exp(rate * softplus(dt_pre + dt_bias))
+//   S <- g S;  u = beta (v - S^T k^);  S <- S + k^ u^T;  o = S^T q^
+// q, k (kv_heads x dim) and v (heads x vdim) are column blocks of one row-major buffer of type t (leading dimension ld); head
+// h uses query/key head h / (heads / kv_heads).  beta_pre, dt_pre: type t, [T, heads] with leading dimension ld_gate; dt_bias,
+// rate: fp32 [heads].  states: fp32 [slot][heads][dim][vdim]; seqs as for gla_scan (a sequence whose first position is 0
+// starts from a zero state).  o: fp32 [T, heads * vdim].
+struct DeltaArgs {
+  const void* qkv; DType t; int ld, q_off, k_off, v_off;
+  const void* beta_pre; const void* dt_pre; int ld_gate;
+  const float* dt_bias; const float* rate;
+  float q_scale, unit_eps;
+  float* states; const int* seqs; int nseq; int T;
+  int heads, kv_heads, dim, vdim;
+  float* o;
+};
+int delta_scan(const DeltaArgs& a, cudaStream_t st);
+
 // ---------------------------------------------------------------- latent attention (latent_attention.cu)
 // Rotation table for interleaved pairs (2i, 2i+1): cs[p][i] = (cos, sin)(p * base^(-2i/dims)), computed in double.
 int rope_table_interleaved(float2* table, int max_pos, int dims, double base, cudaStream_t st);
@@ -254,8 +273,8 @@ int qk_rope_norm_cache(const QkPrepArgs& a, cudaStream_t st);
 // zeros before the sequence's start; conv_w null: no convolution); the convolved keys are the values of the cache row;
 // the whole query row (all heads at once) and the whole key row are divided by their root mean square (eps inside the
 // root) and multiplied by q_norm_w [heads * dim] / k_norm_w [kv_heads * dim]; the first rot_dims dimensions of every head
-// are rotated by the token's position, dimension i paired with i + rot_dims / 2 (rotate-half layout; rope as
-// rope_table_yarn writes it); query head h is multiplied by q_head_scale[h] (optional: a temperature per head).
+// are rotated by the token's position, dimension i paired with i + rot_dims / 2 (rotate-half layout) or, with interleaved,
+// 2i with 2i + 1 (rope as rope_table_yarn writes it, either way); query head h is multiplied by q_head_scale[h] (optional: a temperature per head).
 // Queries go to qn (fp32 [T, heads * dim]), keys to the cache row [kv_heads * dim (keys) | kv_heads * dim (values)].
 // The carried inputs are written afterwards by short_conv_carry over the same columns.
 struct ConvQkPrepArgs {
@@ -267,6 +286,7 @@ struct ConvQkPrepArgs {
   const int* positions; const int* slots; const int* seq_of_tok; const int* seqs;
   float* qn; void* cache;
   int T, heads, kv_heads, dim;
+  bool interleaved = false;
 };
 int conv_qk_prep(const ConvQkPrepArgs& a, cudaStream_t st);
 // Softmax attention of token t (position p of its sequence) over the cached keys j <= p with p - j < window or
@@ -332,6 +352,10 @@ int selective_scan(const SelectiveScanArgs& a, cudaStream_t st);
 // x[s][t] = embed[ids[t]] * scale for every stream s (fp32; stream s starts at x + s * stream_stride).
 int embed_scaled(const void* embed, DType tw, const int* ids, float* x, int T, int W, int vocab, float scale, int streams,
                  long long stream_stride, cudaStream_t st);
+// x[t] = embed[ids[t]] / sqrt(mean(embed[ids[t]]^2) + eps) * w (fp32 [T, W]), and the same row in type th at h (may be null):
+// a residual that starts from normed embeddings, with the row its first sublayer reads.
+int embed_normed(const void* embed, DType tw, const int* ids, const float* w, float eps, float* x, void* h, DType th, int T, int W, int vocab,
+                 cudaStream_t st);
 // One boundary between two sublayers on `streams` fp32 residual streams (1..8).  For r < rows, t = row_index ? row_index[r] : r:
 //   if (y)  all streams at once from the old ones: x_j[t] <- sum_s mix[s * streams + j] * x_s[t] + out[j] * y[t]
 //           (mix null: identity; out null: ones; with one stream and both null this is the plain residual sum)
@@ -398,8 +422,15 @@ enum MoeScore { MOE_SOFTMAX = 0, MOE_SIGMOID = 1, MOE_TOP_SOFTMAX = 2 };
 // ld: leading dimension of scores (0: E); columns past E are left alone (a design may keep other fp32 outputs there).
 // select_bias (optional, fp32 [E]; MOE_SOFTMAX and MOE_SIGMOID): experts (and groups) are ranked by score + select_bias,
 // the weights stay the scores themselves.
+// MoeRouteForm: a group is ranked by the sum of its group_best (1 or 2) largest members; with normalize the weights are the
+// chosen scores divided by their sum + sum_eps and multiplied by scale (MOE_SOFTMAX and MOE_SIGMOID).
+struct MoeRouteForm {
+  int group_best = 1;
+  bool normalize = false;
+  float sum_eps = 0.f, scale = 1.f;
+};
 int moe_route(float* scores, int* topk_ids, float* topk_w, int T, int E, int groups, int keep, int top, cudaStream_t st,
-              int score_fn = MOE_SOFTMAX, int ld = 0, const float* select_bias = nullptr);
+              int score_fn = MOE_SOFTMAX, int ld = 0, const float* select_bias = nullptr, const MoeRouteForm& form = MoeRouteForm());
 // Sort the T * top (token, choice) pairs by expert into 64-row tiles: sorted_rows[cap] = token of each sorted row or -1,
 // tile_group[cap / 64] = expert of each tile or -1, pair_pos[T * top] = sorted row of each pair.  cap >= T*top + E*64.
 // expert_rows (optional): [E][2] = {first sorted row, rows} of every expert.

@@ -115,5 +115,6 @@ std::unique_ptr<Model> make_zinavik(const JVal& config, DType dtype, std::string
 std::unique_ptr<Model> make_mulenex(const JVal& config, DType dtype, std::string* err);
 std::unique_ptr<Model> make_nagilix(const JVal& config, DType dtype, std::string* err);
 std::unique_ptr<Model> make_soselix(const JVal& config, DType dtype, std::string* err);
+std::unique_ptr<Model> make_dabodra(const JVal& config, DType dtype, std::string* err);
 
 }  // namespace b200

@@ -15,6 +15,7 @@ const Entry kModels[] = {
     {"Mulenex", make_mulenex},
     {"Nagilix", make_nagilix},
     {"Soselix", make_soselix},
+    {"Dabodra", make_dabodra},
 };
 }  // namespace
 

@@ -2,8 +2,8 @@
 // pairs into expert-grouped 64-row tiles for the grouped launches of linear.cu, and the weighted combine.
 //
 // Routing of one token: s = softmax(z) over all E experts; the experts form `groups` equal groups of neighbours, a group
-// is ranked by its largest s, only the `keep` best groups stay eligible; the `top` largest eligible s win, ties to the
-// lower index, and s itself (not renormalised) is the weight.  Other forms score by sigmoid(z) alone, or rank by z and
+// is ranked by its largest s (or the sum of its two largest), only the `keep` best groups stay eligible; the `top` largest eligible s win, ties to the
+// lower index, and s itself (or its share of the winners' sum times a constant) is the weight.  Other forms score by sigmoid(z) alone, or rank by z and
 // weight the winners by the softmax over the winners' z only.  A pair's result never depends on which other pairs
 // share its tile, and the combine adds a token's choices in the order the router picked them.
 #include <cuda_bf16.h>
@@ -19,7 +19,7 @@ typedef __nv_bfloat16 bf16;
 
 // one warp per token; scores row in global memory is the scratch (chosen entries are overwritten with -1)
 __global__ void moe_route_kernel(float* scores, int* topk_ids, float* topk_w, int T, int E, int groups, int keep, int top, int score_fn, int ld,
-                                 const float* bias) {
+                                 const float* bias, MoeRouteForm form) {
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (t >= T) return;
   const int lane = threadIdx.x & 31;
@@ -53,8 +53,13 @@ __global__ void moe_route_kernel(float* scores, int* topk_ids, float* topk_w, in
     int bg = 0x7fffffff;
     for (int g = lane; g < groups; g += 32) {
       if (kept >> g & 1ull) continue;
-      float gm = lowest;
-      for (int e = g * per; e < (g + 1) * per; ++e) gm = fmaxf(gm, rank(e));
+      float gm = lowest, second = lowest;
+      for (int e = g * per; e < (g + 1) * per; ++e) {
+        const float v = rank(e);
+        second = fmaxf(second, fminf(gm, v));
+        gm = fmaxf(gm, v);
+      }
+      if (form.group_best == 2 && per > 1) gm += second;
       if (gm > best) { best = gm; bg = g; }
     }
     for (int o = 16; o > 0; o >>= 1) {
@@ -64,7 +69,7 @@ __global__ void moe_route_kernel(float* scores, int* topk_ids, float* topk_w, in
     }
     if (bg != 0x7fffffff) kept |= 1ull << bg;
   }
-  float first = 0.f, sum = 0.f;   // MOE_TOP_SOFTMAX: the largest chosen logit and the sum of exp(logit - first) over the chosen
+  float first = 0.f, sum = 0.f;   // MOE_TOP_SOFTMAX: the largest chosen logit and the sum of exp(logit - first) over the chosen; else the chosen scores' sum
   for (int k = 0; k < top; ++k) {
     float best = lowest;
     int be = 0x7fffffff;
@@ -81,7 +86,7 @@ __global__ void moe_route_kernel(float* scores, int* topk_ids, float* topk_w, in
     if (be == 0x7fffffff) { be = 0; best = 0.f; }
     else if (bias) best = s[be];     // the weight is the score without the bias
     if (k == 0) first = best;
-    sum += expf(best - first);
+    sum += score_fn == MOE_TOP_SOFTMAX ? expf(best - first) : best;
     if (lane == 0) {
       topk_ids[static_cast<long long>(t) * top + k] = be;
       topk_w[static_cast<long long>(t) * top + k] = best;
@@ -94,6 +99,11 @@ __global__ void moe_route_kernel(float* scores, int* topk_ids, float* topk_w, in
     for (int k = lane; k < top; k += 32) {
       float* w = topk_w + static_cast<long long>(t) * top + k;
       *w = expf(*w - first) * inv;
+    }
+  } else if (form.normalize) {
+    for (int k = lane; k < top; k += 32) {
+      float* w = topk_w + static_cast<long long>(t) * top + k;
+      *w = *w / (sum + form.sum_eps) * form.scale;
     }
   }
 }
@@ -159,11 +169,12 @@ __global__ void moe_combine_kernel(const TYIN* y, const int* pair_pos, const flo
 }  // namespace
 
 int moe_route(float* scores, int* topk_ids, float* topk_w, int T, int E, int groups, int keep, int top, cudaStream_t st, int score_fn, int ld,
-              const float* select_bias) {
+              const float* select_bias, const MoeRouteForm& form) {
   if (T <= 0) return 0;
   if (E < 1 || groups < 1 || groups > 64 || E % groups || keep < 1 || keep > groups || top < 1 || top > keep * (E / groups)) return -1;
-  if (select_bias && score_fn == MOE_TOP_SOFTMAX) return -1;
-  moe_route_kernel<<<(T + 3) / 4, 128, 0, st>>>(scores, topk_ids, topk_w, T, E, groups, keep, top, score_fn, ld > 0 ? ld : E, select_bias);
+  if ((select_bias || form.normalize) && score_fn == MOE_TOP_SOFTMAX) return -1;
+  if (form.group_best < 1 || form.group_best > 2) return -1;
+  moe_route_kernel<<<(T + 3) / 4, 128, 0, st>>>(scores, topk_ids, topk_w, T, E, groups, keep, top, score_fn, ld > 0 ? ld : E, select_bias, form);
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
 

@@ -3,8 +3,8 @@
 // frequency scaling and a unit-RMS norm of every query and key head, optionally with a weight, a position-dependent query
 // gain and a blend of the values with an earlier layer's (QkPrepArgs).  Scores may be tanh-capped, the sigmoid output
 // gate is per output column or per head.  A second preparation (ConvQkPrepArgs) serves attention whose queries and keys
-// pass a short causal convolution, a norm over the whole projection and a rotate-half rotation, and whose values are the
-// convolved keys.  Visibility may be chunked instead of windowed (the first visible key is the start of the token's
+// may pass a short causal convolution, then a norm over the whole projection and a rotation of either layout, and whose
+// values are the keys before norm and rotation.  Visibility may be chunked instead of windowed (the first visible key is the start of the token's
 // chunk), and the softmax may have a sink, a learned per-head term exp(sink) of the denominator that belongs to no cached token.
 //
 // Visibility of key j for the token at position p: j <= p and (p - j < window or j < keep_first).  The visible keys of
@@ -116,8 +116,8 @@ __global__ void __launch_bounds__(128) qk_prep_kernel(QkPrepArgs a) {
 // One CTA per token (ConvQkPrepArgs).  Pass 1: a thread per channel convolves the projections over time (its taps come
 // from the step's own rows or from the sequence's carried inputs), leaves the result in shared memory, writes the
 // convolved keys as the values of the cache row and adds to the sum of squares of the query row or of the key row; the two
-// sums meet in shared memory in warp order.  Pass 2: a thread per rotation pair (dimension i with i + rot_dims / 2) or
-// unrotated column normalises over the WHOLE projection, applies the weights, rotates, applies the head's temperature to
+// sums meet in shared memory in warp order.  Pass 2: a thread per rotation pair (dimension i with i + rot_dims / 2, or 2i with
+// 2i + 1) or unrotated column normalises over the WHOLE projection, applies the weights, rotates, applies the head's temperature to
 // queries and writes qn or the key part of the cache row.
 template <typename T>
 __global__ void __launch_bounds__(1024) conv_qk_prep_kernel(ConvQkPrepArgs a) {
@@ -175,18 +175,19 @@ __global__ void __launch_bounds__(1024) conv_qk_prep_kernel(ConvQkPrepArgs a) {
     const int u_ = it / per_head, k = it - u_ * per_head;
     const bool isq = u_ < a.heads;
     const int hd = isq ? u_ : u_ - a.heads;
-    const int cc = hd * D + (k < half ? k : k + half);     // column within the query or the key row
+    const int c1 = a.interleaved ? 2 * k : k, step = a.interleaved ? 1 : half;   // first column of the pair, distance to its second
+    const int cc = hd * D + (k < half ? c1 : k + half);     // column within the query or the key row
     const float inv = isq ? invq : invk;
     const float* nwt = isq ? a.q_norm_w : a.k_norm_w;
     const float* row = cv + (isq ? 0 : HD);
     const float hs = (isq && a.q_head_scale) ? a.q_head_scale[hd] : 1.0f;
     const float lo = row[cc] * inv * (nwt ? nwt[cc] : 1.0f);
     if (k < half) {
-      const float hi = row[cc + half] * inv * (nwt ? nwt[cc + half] : 1.0f);
+      const float hi = row[cc + step] * inv * (nwt ? nwt[cc + step] : 1.0f);
       const float2 r = cs[k];
       const float o0 = lo * r.x - hi * r.y, o1 = hi * r.x + lo * r.y;
-      if (isq) { a.qn[t * HD + cc] = o0 * hs; a.qn[t * HD + cc + half] = o1 * hs; }
-      else { stf(cache + cc, o0); stf(cache + cc + half, o1); }
+      if (isq) { a.qn[t * HD + cc] = o0 * hs; a.qn[t * HD + cc + step] = o1 * hs; }
+      else { stf(cache + cc, o0); stf(cache + cc + step, o1); }
     } else {
       if (isq) a.qn[t * HD + cc] = lo * hs;
       else stf(cache + cc, lo);
