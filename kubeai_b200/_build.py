@@ -30,6 +30,7 @@ SOURCES = [
     "gla.cu",
     "scan_chunk.cu",
     "delta.cu",
+    "delta_chunk.cu",
     "latent_attention.cu",
     "moe.cu",
     "hyper.cu",

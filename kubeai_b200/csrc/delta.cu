@@ -151,6 +151,12 @@ int delta_scan(const DeltaArgs& a, cudaStream_t st) {
   if (a.nseq <= 0 || a.T <= 0) return 0;
   if (!a.qkv || !a.beta_pre || !a.dt_pre || !a.dt_bias || !a.rate || !a.states || !a.seqs || !a.o || a.heads < 1 || a.kv_heads < 1 ||
       a.heads % a.kv_heads || a.dim < 1 || a.vdim < 1) return -1;
+  if (delta_chunk_fits(a)) {
+    // steps that bring portions (B200_DELTA_CHUNK: A/B knob, the mean portion from which the chunked form runs; 0 = never)
+    const char* e = getenv("B200_DELTA_CHUNK");
+    const int from = e ? atoi(e) : 8;
+    if (from > 0 && a.T >= static_cast<long long>(from) * a.nseq) return delta_chunk(a, st);
+  }
   int P = 1;
   while (P * 4 * kPieces < a.dim) P <<= 1;
   if (P > 32) return -1;   // dim <= 1024

@@ -198,6 +198,10 @@ struct DeltaArgs {
   float* o;
 };
 int delta_scan(const DeltaArgs& a, cudaStream_t st);
+// The chunked tensor-core form of the same scan (delta_chunk.cu; same result up to fp32 rounding), for the shapes it takes;
+// delta_scan chooses it for bf16 steps of prompt portions.
+bool delta_chunk_fits(const DeltaArgs& a);
+int delta_chunk(const DeltaArgs& a, cudaStream_t st);
 
 // ---------------------------------------------------------------- latent attention (latent_attention.cu)
 // Rotation table for interleaved pairs (2i, 2i+1): cs[p][i] = (cos, sin)(p * base^(-2i/dims)), computed in double.

@@ -4,7 +4,8 @@ and feed-forward sizes, on random weights (`bench.py --design nomanex`: beside t
 kernels; `bench.py --design mulenex`: beside Zinavik, which runs the same attention, scan, routing and projection kernels;
 `bench.py --design nagilix`: beside Zinavik, whose streams, paged attention, constant-decay scan and clamped routed experts
 are the like kernels; `bench.py --design soselix`: beside Nomanex with dense feed-forwards in every layer, whose latent
-attention, recurrent scan and projections are the like kernels).  Every number is CUDA-event time of the engine's
+attention, recurrent scan and projections are the like kernels; `bench.py --design dabodra`: beside Mulenex with routed experts
+in every layer, whose boundaries with output norms, paged attention, recurrent scan and expert kernels are the like ones).  Every number is CUDA-event time of the engine's
 own step (b200_feed_step: the same packing, page pool, state slots and kernels as a scheduled step), after warm-up
 steps, with a buffer larger than L2 written between timed steps.  Per-kernel times come from a separate pass in which
 each launch is bracketed by events (b200_engine_profile_kernels for the design, b200_engine_profile_range for Llama),
@@ -80,6 +81,23 @@ def soselix_config(z):
     layers = [dict(type="latent_attention", mixer=la, mlp=dn), dict(type="hgrn2", mixer=hg, mlp=dn), dict(type="mamba2", mixer=ma, mlp=dn),
               dict(type="latent_attention", mixer=dict(la, kv_from=0), mlp=dn)]
     return dict(architecture="Soselix", vocab=z["vocab"], width=W, residual_mult=0.5, norm=dict(eps=1e-5), embedding=dict(scale=1.0), layers=layers)
+
+
+def dabodra_config(z):
+    H = z["heads"]
+    at = dict(heads=H, kv_heads=max(1, H // 4), dim=DIM, vdim=DIM, mask=dict(size=z["window"]), rot=dict(base=10000.0, dims=ROT), scale=DIM ** -0.5)
+    de = dict(heads=H, kv_heads=H, dim=DIM, vdim=VDIM, conv=4)
+    mo = dict(kind="moe", expert=dict(ff=z["eff"]), router=dict(experts=z["experts"], top=z["top"], groups=dict(count=z["groups"], keep=z["keep"]), scale=1.0),
+              shared=dict(ff=z["eff"]))
+    la, ld = dict(type="attention", mixer=at, mlp=mo), dict(type="delta", mixer=de, mlp=mo)
+    return dict(architecture="Dabodra", vocab=z["vocab"], width=z["width"], norm=dict(eps=1e-5), layers=[la, ld, la, ld])
+
+
+def mulenex_moe_config(z):
+    c = mulenex_config(z)
+    for ly in c["layers"]:
+        ly["mlp"] = c["layers"][0]["mlp"]
+    return c
 
 
 def nomanex_dense_config(z):
@@ -200,6 +218,32 @@ def run_design(cfgj, lim, z, batch, prompt, decode_steps, warmup, peaks, torch, 
                     "mamba2_gate_norm_prefill_frac_of_hbm": T * Hm * P * (4 + 2 + 2 + 2.0) / us(kp, "mamba2_gate_norm") / (hbm * 1e9),
                     "hgrn2_out_norm_prefill_frac_of_hbm": T * H * VDIM * (4 + 2.0) / us(kp, "hgrn2_out_norm") / (hbm * 1e9),
                 }
+            elif cfgj["architecture"] == "Dabodra":
+                att = [ly for ly in cfgj["layers"] if ly["type"] == "attention"]
+                rec = [ly for ly in cfgj["layers"] if ly["type"] == "delta"]
+                L, La, Ld = len(cfgj["layers"]), len(att), len(rec)
+                G, Gd, win = att[0]["mixer"]["kv_heads"], rec[0]["mixer"]["kv_heads"], att[0]["mixer"]["mask"]["size"]
+                keys = sum(min(p + 1, win) for p in range(prompt)) * batch
+                conv_c = 2 * Gd * DIM + H * VDIM
+                n_in = La * (H + G) * DIM + Ld * (conv_c + H * VDIM + 2 * H)
+                k_out = La * H * DIM + Ld * H * VDIM
+                dkeys = batch * min(prompt + 1, win)
+                calls = 2 * L
+                r["roofline"] = {
+                    "attention_prefill_frac_of_bf16_peak": 2.0 * La * H * keys * 2 * DIM / us(kp, "window_attention") / (tf * 1e12),
+                    "delta_scan_prefill_tflops": 6.0 * Ld * T * H * DIM * VDIM / us(kp, "delta_scan") / 1e12,
+                    "projections_prefill_frac_of_bf16_peak": 2.0 * T * W * (n_in + k_out) / (us(kp, "proj_in") + us(kp, "proj_out")) / (tf * 1e12),
+                    "delta_scan_decode_frac_of_hbm": 2.0 * Ld * batch * H * DIM * VDIM * 4 / us(kd, "delta_scan") / (hbm * 1e9),
+                    "attention_decode_frac_of_hbm": La * dkeys * G * 2 * DIM * 2.0 / us(kd, "window_attention") / (hbm * 1e9),
+                    "projections_decode_frac_of_hbm": 2.0 * W * (n_in + k_out) / (us(kd, "proj_in") + us(kd, "proj_out")) / (hbm * 1e9),
+                    # boundary: reads and writes the fp32 residual, reads a bf16 sublayer output, writes a bf16 row
+                    "residual_norm_prefill_frac_of_hbm": calls * T * W * (8.0 + 2 + 2) / us(kp, "residual_norm") / (hbm * 1e9),
+                    # preparation: reads the q | k row, writes fp32 queries and the cache row
+                    "qk_prep_prefill_frac_of_hbm": La * T * ((H + G) * DIM * 2.0 + H * DIM * 4 + 2 * G * DIM * 2) / us(kp, "qk_prep") / (hbm * 1e9),
+                    "short_conv_prefill_frac_of_hbm": Ld * T * conv_c * 4.0 / us(kp, "short_conv") / (hbm * 1e9),
+                    "delta_out_gate_prefill_frac_of_hbm": Ld * T * H * VDIM * (4.0 + 2 + 2) / us(kp, "delta_out_gate") / (hbm * 1e9),
+                    **_moe_roofline(z, L, T, batch, W, kp, kd, us, hbm, tf),
+                }
             elif cfgj["architecture"] == "Nagilix":
                 par = [ly for ly in cfgj["layers"] if ly["type"] == "parallel"]
                 mam = [ly for ly in cfgj["layers"] if ly["type"] == "mamba1"]
@@ -261,10 +305,11 @@ def run_design(cfgj, lim, z, batch, prompt, decode_steps, warmup, peaks, torch, 
                     "projections_decode_frac_of_hbm": 2.0 * W * (n_in + k_out) / (us(kd, "proj_in") + us(kd, "proj_out")) / (hbm * 1e9),
                     # boundary: reads and writes the fp32 residual, reads a bf16 sublayer output, writes a bf16 row
                     "residual_norm_prefill_frac_of_hbm": calls * T * W * (8.0 + 2 + 2) / us(kp, "residual_norm") / (hbm * 1e9),
-                    "moe_experts_prefill_frac_of_bf16_peak": 2.0 * moes * T * z["top"] * 3 * W * z["eff"] / (us(kp, "moe_up") + us(kp, "moe_down")) / (tf * 1e12),
-                    "dense_ff_prefill_frac_of_bf16_peak": 2.0 * T * 2 * W * z["ff"] / (us(kp, "ff_up") + us(kp, "ff_down")) / (tf * 1e12),
+                    **({"dense_ff_prefill_frac_of_bf16_peak": 2.0 * T * 2 * W * z["ff"] / (us(kp, "ff_up") + us(kp, "ff_down")) / (tf * 1e12)} if "ff_up" in kp else {}),
                     # gate chain, out gate: the small kernels around the scan, as time beside the scan's
                     "mlstm_gates_prefill_us": us(kp, "mlstm_gates") * 1e6 + us(kp, "mlstm_gate_proj") * 1e6,
+                    "qk_prep_prefill_frac_of_hbm": len(att) * T * ((H * DIM + G * (DIM + VDIM)) * 2.0 + H * DIM * 4 + G * (DIM + VDIM) * 2) / us(kp, "qk_prep") / (hbm * 1e9),
+                    **_moe_roofline(z, moes, T, batch, W, kp, kd, us, hbm, tf),
                     "mlstm_out_gate_prefill_frac_of_hbm": len(rec) * T * H * ((VDIM + 1) * 4.0 + VDIM * 2 + VDIM * 2) / us(kp, "mlstm_out_gate") / (hbm * 1e9),
                 }
             else:
@@ -294,6 +339,21 @@ def run_design(cfgj, lim, z, batch, prompt, decode_steps, warmup, peaks, torch, 
     return r
 
 
+def _moe_roofline(z, layers, T, batch, W, kp, kd, us, hbm, tf):
+    """Routed experts and the shared expert (three matrices each), and the rows their elementwise kernels move."""
+    F, top = z["eff"], z["top"]
+    return {
+        "moe_experts_prefill_frac_of_bf16_peak": 2.0 * layers * T * top * 3 * W * F / (us(kp, "moe_up") + us(kp, "moe_down")) / (tf * 1e12),
+        "shared_expert_prefill_frac_of_bf16_peak": 2.0 * layers * T * 3 * W * F / (us(kp, "shared_in") + us(kp, "shared_down")) / (tf * 1e12),
+        # decode: every chosen (token, expert) pair streams its expert's weights (pairs that share an expert read it from L2)
+        "moe_experts_decode_frac_of_hbm": 2.0 * layers * min(batch * top, z["experts"]) * 3 * W * F / (us(kd, "moe_up") + us(kd, "moe_down")) / (hbm * 1e9),
+        "shared_expert_decode_frac_of_hbm": 2.0 * layers * 3 * W * F / (us(kd, "shared_in") + us(kd, "shared_down")) / (hbm * 1e9),
+        "glu_prefill_frac_of_hbm": layers * T * (top + 1) * F * 6.0 / us(kp, "glu") / (hbm * 1e9),
+        "moe_combine_prefill_frac_of_hbm": layers * T * W * 2.0 * (top + 2) / us(kp, "moe_combine") / (hbm * 1e9),
+        "moe_route_prefill_us": (us(kp, "moe_router") + us(kp, "moe_route") + us(kp, "moe_align") + us(kp, "moe_gather")) * 1e6,
+    }
+
+
 def bench_size(design, name, z, batch, prompt, decode_steps, warmup, peaks):
     import torch
     from .engine import Engine, default_config
@@ -304,6 +364,11 @@ def bench_size(design, name, z, batch, prompt, decode_steps, warmup, peaks):
     lim["num_kv_blocks"] = batch * ((lim["max_model_len"] + 15) // 16)
     res = {"size": dict(z, batch=batch, prompt=prompt)}
     T = batch * prompt
+    if design == "dabodra":
+        res["dabodra"] = run_design(dabodra_config(z), lim, z, batch, prompt, decode_steps, warmup, peaks, torch, buf)
+        res["mulenex"] = run_design(mulenex_moe_config(z), lim, z, batch, prompt, decode_steps, warmup, peaks, torch, buf)
+        del buf
+        return res
     if design == "soselix":
         res["soselix"] = run_design(soselix_config(z), lim, z, batch, prompt, decode_steps, warmup, peaks, torch, buf)
         res["nomanex"] = run_design(nomanex_dense_config(z), lim, z, batch, prompt, decode_steps, warmup, peaks, torch, buf)
@@ -371,8 +436,9 @@ def _k_out(ly):
 
 
 def run(design, peaks, sizes=None, batch=8, prompt=512, decode_steps=8, warmup=3):
-    if design not in ("nomanex", "zinavik", "mulenex", "nagilix", "soselix"):
-        raise SystemExit("unknown design %r (known: nomanex, zinavik, mulenex, nagilix, soselix)" % design)
+    known = ("nomanex", "zinavik", "mulenex", "nagilix", "soselix", "dabodra")
+    if design not in known:
+        raise SystemExit("unknown design %r (known: %s)" % (design, ", ".join(known)))
     out = {"design": design, "dtype": "bf16", "data": "synthetic (seeded random weights and tokens)", "peaks": dict(hbm_gbs=peaks[0], bf16_tflops=peaks[1], source=peaks[2]),
            "timing": "CUDA events around the engine step, median of the timed steps, %d warm-up steps, 320 MB written between steps" % warmup,
            "sizes": {}}

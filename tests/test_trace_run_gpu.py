@@ -9,6 +9,7 @@ import sys
 import numpy as np
 import pytest
 
+import dabodra_util as dx
 import mulenex_util as mx
 import nagilix_util as nx
 import soselix_util as sx
@@ -75,8 +76,16 @@ def soselix_model():
     return cfg, W, sx.oracle_for(cfg, W)
 
 
+def dabodra_model():
+    layers = [dx.attention(heads=6, kv_heads=3, dim=16, window=21, rot_dims=8, mlp=dx.moe(experts=4, top=4, count=2, keep=2, ff=24, shared=8)),
+              dx.delta(heads=4, kv_heads=2, dim=16, vdim=24, conv=5, mlp=None), dx.attention(heads=2, kv_heads=2, dim=8, window=50, mlp=None)]
+    cfg = dx.make_config(layers, width=40, vocab=70)
+    W = dx.random_weights(cfg, seed=99)
+    return cfg, W, dx.oracle_for(cfg, W)
+
+
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("model", [zinavik_model, mulenex_model, nagilix_model, soselix_model])
+@pytest.mark.parametrize("model", [zinavik_model, mulenex_model, nagilix_model, soselix_model, dabodra_model])
 def test_replayed_schedule_gives_the_oracles_logits(tmp_path, dtype, model):
     cfg, W, o = model()
     d = write_model_dir(tmp_path / "m", cfg, W)
