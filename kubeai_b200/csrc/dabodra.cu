@@ -73,14 +73,17 @@ struct LayerWeights {
   float *conv_w = nullptr, *dt_b = nullptr, *rate = nullptr, *o_norm = nullptr;   // delta: [conv_c, taps], [heads], [heads] (-exp(A_log)), [vdim]
   void* router = nullptr;   // [experts, width]
   float* correction = nullptr;
-  void* e_gu = nullptr;     // [experts][2 ff][width]  gate rows, then up rows
+  void* e_gu = nullptr;     // [experts][2 ff][width]  gate rows, then up rows (or in turns, see il_e)
   void* e_down = nullptr;   // [experts][width][ff]
-  void* sh_in = nullptr;    // [n_sh, width]: gate [sff] | up [sff]
+  void* sh_in = nullptr;    // [n_sh, width]: gate [sff] | up [sff] (or in turns, see il_s)
   void* sh_down = nullptr;  // [width, sff]
   GemmPlan p_in, p_out, p_shin, p_shdown;
-  std::vector<GemmPlan> p_egu, p_edown;
+  GroupedPlan g_egu, g_edown;
+  CUtensorMap xg_h, xg_act;                                    // the grouped form's views of the sorted rows and of the hidden rows
   CUtensorMap xm_out[kGemmNumBlockN], xm_shact[kGemmNumBlockN];
-  bool tc_in = false, tc_out = false, tc_shin = false, tc_shdown = false;
+  bool tc_in = false, tc_out = false, tc_shin = false, tc_shdown = false, tc_experts = false;
+  // gate and up rows in alternating blocks of 64, so that one GEMM tile holds both and its epilogue can join them
+  bool il_e = false, il_s = false;
 };
 
 struct LayerRun {
@@ -112,7 +115,8 @@ class Dabodra : public Model {
   void *h = nullptr, *inb = nullptr, *xc = nullptr, *yb = nullptr, *ao = nullptr, *fo = nullptr, *hrow = nullptr;
   void *egu = nullptr, *eact = nullptr, *sh = nullptr, *shact = nullptr, *sdown = nullptr, *hsorted = nullptr, *edown16 = nullptr;
   int *topi = nullptr, *sorted_rows = nullptr, *tile_group = nullptr, *pair_pos = nullptr, *iota = nullptr;
-  int *expert_rows = nullptr, *expert_rows_host = nullptr;
+  int* expert_rows = nullptr;
+  int* kernel_error = nullptr;   // pinned: a kernel whose wait ran out leaves a mark here
   int row_cap = 0, moe_cap = 0;
   std::vector<void*> allocs;
   float* gemm_ws = nullptr;
@@ -120,7 +124,7 @@ class Dabodra : public Model {
   int* gemm_flags = nullptr;     // of the fused form: two per CTA pair, stamped with the launch's number
   int gemm_epoch = 0;
   bool fuse = true;
-  int few_rows = 16, moe_tc_min = 256;
+  int few_rows = 16;
   CUtensorMap xm_h[kGemmNumBlockN];
   bool use_tc = false;
 
@@ -131,11 +135,9 @@ class Dabodra : public Model {
       if (w.tc_out) gemm_plan_destroy(&w.p_out);
       if (w.tc_shin) gemm_plan_destroy(&w.p_shin);
       if (w.tc_shdown) gemm_plan_destroy(&w.p_shdown);
-      for (auto& p : w.p_egu) gemm_plan_destroy(&p);
-      for (auto& p : w.p_edown) gemm_plan_destroy(&p);
     }
     if (pe0) { cudaEventDestroy(pe0); cudaEventDestroy(pe1); }
-    if (expert_rows_host) cudaFreeHost(expert_rows_host);
+    if (kernel_error) cudaFreeHost(kernel_error);
     for (void* p : allocs) cudaFree(p);
   }
   const char* arch() const override { return "Dabodra"; }
@@ -321,6 +323,8 @@ class Dabodra : public Model {
       const LayerSpec& s = spec[i];
       LayerWeights& w = wts[i];
       LayerRun& r = run[i];
+      w.il_e = dt == DT_BF16 && s.mlp && s.ff % 64 == 0;
+      w.il_s = dt == DT_BF16 && s.shared && s.sff % 64 == 0;
       rc |= mat(&w.w_in, s.n_in, W) | mat(&w.w_out, W, s.k_out) | vec(&w.norm1, W);
       if (s.kind == MIX_ATTENTION) {
         rc |= vec(&w.q_norm, static_cast<size_t>(s.heads) * s.dim) | vec(&w.k_norm, static_cast<size_t>(s.kv_heads) * s.dim) | vec(&w.sink, s.heads) |
@@ -347,6 +351,8 @@ class Dabodra : public Model {
     if (max_rec) rc |= mat(&xc, T, max_xc) | vec(&o32, T * max_rec);
     if (any_moe) {
       moe_cap = static_cast<int>((T * max_top + 63) / 64 * 64) + max_e * 64;
+      if (cudaMallocHost(&kernel_error, sizeof(int)) != cudaSuccess) return -3;
+      *kernel_error = 0;
       rc |= mat(&fo, T, W) | vec(&scores, T * max_e) | vec(&topw, T * max_top) | dalloc(&topi, T * max_top * sizeof(int)) |
             dalloc(&sorted_rows, static_cast<size_t>(moe_cap) * sizeof(int)) | dalloc(&tile_group, static_cast<size_t>(moe_cap / 64) * sizeof(int)) |
             dalloc(&pair_pos, T * max_top * sizeof(int)) | mat(&egu, moe_cap, 2 * static_cast<size_t>(max_ff)) | mat(&eact, moe_cap, max_ff) |
@@ -366,8 +372,8 @@ class Dabodra : public Model {
   }
 
   // The projections of a bf16 model run on the tcgen05 pair GEMM (gemm2_tcgen05.cu) where their shapes allow it (rows and
-  // columns in multiples of 8): input and output projection, the shared expert, and every expert for steps large enough to
-  // sort rows per expert.  B200_DB_TC=0 keeps everything on linear.cu (A/B knob); fp32 models always do.
+  // columns in multiples of 8): input and output projection and the shared expert; the routed experts on its grouped form
+  // (gemm_grouped.cu).  B200_DB_TC=0 keeps everything on linear.cu (A/B knob); fp32 models always do.
   int setup_tc() {
     const char* ev = getenv("B200_DB_TC");
     use_tc = dt == DT_BF16 && !(ev && atoi(ev) == 0) && W % 8 == 0 && gemm_variant() == 2;
@@ -380,7 +386,8 @@ class Dabodra : public Model {
     if (dalloc(&gemm_counters, n_counters * sizeof(int)) || dalloc(&gemm_flags, static_cast<size_t>(env.sms) * 2 * sizeof(int))) return -3;
     if (const char* e = getenv("B200_DB_FUSE")) fuse = atoi(e) != 0;              // A/B knobs
     if (const char* e = getenv("B200_DB_FEW_ROWS")) few_rows = atoi(e);
-    if (const char* e = getenv("B200_DB_MOE_TC_MIN_T")) moe_tc_min = atoi(e);
+    bool grouped = true;
+    if (const char* e = getenv("B200_DB_GROUPED")) grouped = atoi(e) != 0;
     const int bns[kGemmNumBlockN] = {32, 64, 128, 256, 512};
     auto maps = [&](CUtensorMap* m, const void* X, int K) {
       for (int i = 0; i < kGemmNumBlockN; ++i)
@@ -399,7 +406,12 @@ class Dabodra : public Model {
       return false;
     };
     if (!maps(xm_h, h, W)) { use_tc = false; return 0; }
-    int max_e = 0;
+    int max_e = 1;
+    bool any_mlp = false;
+    for (auto& s : spec)
+      if (s.mlp) { any_mlp = true; max_e = std::max(max_e, s.experts); }
+    if (any_mlp && (dalloc(&hsorted, static_cast<size_t>(moe_cap) * W * 2) || dalloc(&edown16, static_cast<size_t>(moe_cap) * W * 2) ||
+                    dalloc(&expert_rows, static_cast<size_t>(max_e) * 2 * sizeof(int)))) return -3;
     for (size_t i = 0; i < spec.size(); ++i) {
       const LayerSpec& s = spec[i];
       LayerWeights& w = wts[i];
@@ -409,25 +421,9 @@ class Dabodra : public Model {
         w.tc_shin = plan(&w.p_shin, w.sh_in, s.n_sh, W);
         w.tc_shdown = plan_maps(&w.p_shdown, w.xm_shact, shact, w.sh_down, W, s.sff);
       }
-      if (!s.mlp || s.ff % 8) continue;
-      bool ok = true;
-      for (int e = 0; e < s.experts && ok; ++e) {
-        GemmPlan gu, dn;
-        ok = plan(&gu, static_cast<bf16*>(w.e_gu) + static_cast<size_t>(e) * 2 * s.ff * W, 2 * s.ff, W);
-        if (!ok) break;
-        w.p_egu.push_back(gu);
-        ok = plan(&dn, static_cast<bf16*>(w.e_down) + static_cast<size_t>(e) * W * s.ff, W, s.ff);
-        if (ok) w.p_edown.push_back(dn);
-      }
-      if (ok) { max_e = std::max(max_e, s.experts); continue; }
-      for (auto& p : w.p_egu) gemm_plan_destroy(&p);
-      for (auto& p : w.p_edown) gemm_plan_destroy(&p);
-      w.p_egu.clear(); w.p_edown.clear();
-    }
-    if (max_e) {
-      if (dalloc(&hsorted, static_cast<size_t>(moe_cap) * W * 2) || dalloc(&edown16, static_cast<size_t>(moe_cap) * W * 2) ||
-          dalloc(&expert_rows, static_cast<size_t>(max_e) * 2 * sizeof(int))) return -3;
-      if (cudaMallocHost(&expert_rows_host, static_cast<size_t>(max_e) * 2 * sizeof(int)) != cudaSuccess) return -3;
+      if (s.mlp && grouped)
+        w.tc_experts = !gemm_grouped_plan(&w.g_egu, w.e_gu, s.experts, 2 * s.ff, W) && !gemm_grouped_plan(&w.g_edown, w.e_down, s.experts, W, s.ff) &&
+                       !gemm_grouped_x_map(&w.xg_h, hsorted, moe_cap, W) && !gemm_grouped_x_map(&w.xg_act, eact, moe_cap, s.ff);
     }
     return 0;
   }
@@ -456,6 +452,17 @@ class Dabodra : public Model {
     }
     return cudaMemcpy(static_cast<uint8_t*>(dst) + row0 * cols * es, tmp.data(), tmp.size(), cudaMemcpyHostToDevice) == cudaSuccess ? 0 : -2;
   }
+  // gate and up rows [F, cols] each, one below the other or in alternating blocks of 64
+  int put_pair(void* dst, size_t row0, const std::vector<float>& gate, const std::vector<float>& up, size_t F, size_t cols, bool in_turns) {
+    std::vector<float> both;
+    both.reserve(2 * F * cols);
+    const size_t block = (in_turns ? 64 : F) * cols;
+    for (size_t at = 0; at < F * cols; at += block) {
+      both.insert(both.end(), gate.begin() + at, gate.begin() + at + block);
+      both.insert(both.end(), up.begin() + at, up.begin() + at + block);
+    }
+    return put(dst, row0, both, 2 * F, cols);
+  }
   int putf(float* dst, const std::vector<float>& src) {
     return cudaMemcpy(dst, src.data(), src.size() * sizeof(float), cudaMemcpyHostToDevice) == cudaSuccess ? 0 : -2;
   }
@@ -476,6 +483,8 @@ class Dabodra : public Model {
     };
     int rc = 0;
 #define MAT(name, dst, row0, rows, cols) do { if (!get(name, rows, cols)) return -4; rc |= put(dst, row0, v, rows, cols); } while (0)
+#define PAIR(prefix, dst, row0, F, cols, turns) do { if (!get((prefix) + "gate", F, cols)) return -4; const std::vector<float> g_ = v; \
+    if (!get((prefix) + "up", F, cols)) return -4; rc |= put_pair(dst, row0, g_, v, F, cols, turns); } while (0)
 #define VEC(name, dst, n) do { if (!get(name, 1, n)) return -4; rc |= putf(dst, v); } while (0)
 #define NORM(name, dst, n) do { if (!get(name, 1, n)) return -4; for (auto& e_ : v) e_ += 1.0f; rc |= putf(dst, v); } while (0)   // stored as the offset from one
     MAT("embed", embed, 0, V, W);
@@ -521,17 +530,16 @@ class Dabodra : public Model {
       VEC(f + "correction", w.correction, s.experts);
       for (int e = 0; e < s.experts; ++e) {
         const std::string ep = f + "e" + std::to_string(e) + ".";
-        MAT(ep + "gate", w.e_gu, static_cast<size_t>(e) * 2 * s.ff, s.ff, W);
-        MAT(ep + "up", w.e_gu, static_cast<size_t>(e) * 2 * s.ff + s.ff, s.ff, W);
+        PAIR(ep, w.e_gu, static_cast<size_t>(e) * 2 * s.ff, s.ff, W, w.il_e);
         MAT(ep + "down", w.e_down, static_cast<size_t>(e) * W, W, s.ff);
       }
       if (s.shared) {
-        MAT(f + "shared.gate", w.sh_in, 0, s.sff, W);
-        MAT(f + "shared.up", w.sh_in, s.sff, s.sff, W);
+        PAIR(f + "shared.", w.sh_in, 0, s.sff, W, w.il_s);
         MAT(f + "shared.down", w.sh_down, 0, W, s.sff);
       }
     }
 #undef MAT
+#undef PAIR
 #undef VEC
 #undef NORM
     if (rc) { *err = "copying weights to the device failed"; return -2; }
@@ -573,17 +581,23 @@ class Dabodra : public Model {
   // ------------------------------------------------------------ forward
   // Y = X W^T.  Steps of up to 16 tokens stream the weights through linear.cu's fragment kernel.  Larger steps take the pair
   // GEMM, in its fused form (whole 256-row tiles, at least one tile per CTA pair) or in its plain one.
+  bool takes_fused(const GemmPlan& plan, bool tc, int T, int N) const {
+    const int bn = block_n(plan, T);
+    return tc && T > few_rows && fuse && N % 256 == 0 && T > 128 && N / 256 * ((T + bn - 1) / bn) >= plan.max_ctas / 2;
+  }
+  int run_fused(const GemmPlan& plan, const CUtensorMap* xm, int epi, void* Y, int ldy, int T) {
+    const int bn = block_n(plan, T);
+    Gemm2Epi e;
+    memset(&e, 0, sizeof(e));
+    e.epi = epi;
+    e.out = static_cast<bf16*>(Y); e.ldo = ldy;
+    e.flags = gemm_flags; e.epoch = ++gemm_epoch;
+    return gemm2_run_fused(plan, xm[gemm_block_n_index(bn)], bn, T, e, env.stream);
+  }
   int project(const GemmPlan& plan, bool tc, const CUtensorMap* xm, const void* X, const void* Wm, void* Y, int T, int N, int K) {
     if (tc && T > few_rows) {
+      if (takes_fused(plan, tc, T, N)) return run_fused(plan, xm, GEMM3_EPI_PLAIN, Y, N, T);
       const int bn = block_n(plan, T);
-      if (fuse && N % 256 == 0 && T > 128 && N / 256 * ((T + bn - 1) / bn) >= plan.max_ctas / 2) {
-        Gemm2Epi e;
-        memset(&e, 0, sizeof(e));
-        e.epi = GEMM3_EPI_PLAIN;
-        e.out = static_cast<bf16*>(Y); e.ldo = N;
-        e.flags = gemm_flags; e.epoch = ++gemm_epoch;
-        return gemm2_run_fused(plan, xm[gemm_block_n_index(bn)], bn, T, e, env.stream);
-      }
       return gemm_run(plan, xm[gemm_block_n_index(bn)], bn, Y, N, T, env.stream);
     }
     return linear(linear_args(X, dt, Wm, dt, Y, dt, T, N, K), env.stream);
@@ -691,20 +705,23 @@ class Dabodra : public Model {
     KRN("moe_route", moe_route(scores, topi, topw, T, s.experts, s.groups, s.keep, s.top, st, MOE_SIGMOID, s.experts, w.correction, form));
     const void* shared_out = nullptr;
     if (s.shared) {
-      KRN("shared_in", project(w.p_shin, w.tc_shin, xm_h, h, w.sh_in, sh, T, s.n_sh, W));
-      KRN("glu", glu_clamped(sh, s.n_sh, shact, s.sff, dt, T, s.sff, INFINITY, 1.f, st, 0.f));
+      if (w.il_s && s.n_sh == 2 * s.sff && takes_fused(w.p_shin, w.tc_shin, T, s.n_sh)) {
+        KRN("shared_in", run_fused(w.p_shin, xm_h, GEMM3_EPI_SILU, shact, s.sff, T));     // the gated unit in the epilogue
+      } else {
+        KRN("shared_in", project(w.p_shin, w.tc_shin, xm_h, h, w.sh_in, sh, T, s.n_sh, W));
+        KRN("glu", glu_clamped(sh, s.n_sh, shact, s.sff, dt, T, s.sff, INFINITY, 1.f, st, 0.f, w.il_s));
+      }
       KRN("shared_down", project(w.p_shdown, w.tc_shdown, w.xm_shact, shact, w.sh_down, sdown, T, W, s.sff));
       shared_out = sdown;
     }
     const long long gu_stride = 2ll * s.ff * W, down_stride = static_cast<long long>(W) * s.ff;
-    const bool per_expert = !w.p_egu.empty() && T >= moe_tc_min;
     if (T * s.top <= 64) {
       // decode-sized steps: one weight-streaming pass per chosen (token, expert) pair, rows in pair order
       LinearArgs up = linear_args(h, dt, w.e_gu, dt, egu, dt, T * s.top, 2 * s.ff, W);
       up.wbs = gu_stride;
       const PickedRows pu = {T * s.top, nullptr, s.top, iota, topi};
       KRN("moe_up", linear_picked_rows(up, pu, st));
-      KRN("glu", glu_clamped(egu, 2 * s.ff, eact, s.ff, dt, T * s.top, s.ff, INFINITY, 1.f, st, 0.f));
+      KRN("glu", glu_clamped(egu, 2 * s.ff, eact, s.ff, dt, T * s.top, s.ff, INFINITY, 1.f, st, 0.f, w.il_e));
       LinearArgs dn = linear_args(eact, dt, w.e_down, dt, edown, DT_F32, T * s.top, W, s.ff);
       dn.wbs = down_stride;
       const PickedRows pd = {T * s.top, iota, 1, iota, topi};
@@ -714,39 +731,24 @@ class Dabodra : public Model {
       return rc;
     }
     const int cap = (T * s.top + 63) / 64 * 64 + s.experts * 64;
-    KRN("moe_align", moe_align(topi, T, s.top, s.experts, sorted_rows, tile_group, pair_pos, cap, st, per_expert ? expert_rows : nullptr));
-    if (per_expert) {
-      // Large steps: every expert's rows are one tcgen05 GEMM.  The row counts come back to the host (one small copy and a
-      // wait per layer, paid only by steps of hundreds of tokens); the inputs are gathered into sorted order.
+    KRN("moe_align", moe_align(topi, T, s.top, s.experts, sorted_rows, tile_group, pair_pos, cap, st, w.tc_experts ? expert_rows : nullptr));
+    if (w.tc_experts) {
+      // the inputs in expert-sorted order, then one grouped GEMM per matrix; the row counts stay on the device
       KRN("moe_gather", moe_gather_bf16(h, sorted_rows, hsorted, cap, W, st));
-      if (cudaMemcpyAsync(expert_rows_host, expert_rows, static_cast<size_t>(s.experts) * 2 * sizeof(int), cudaMemcpyDeviceToHost, st) != cudaSuccess ||
-          cudaStreamSynchronize(st) != cudaSuccess) rc = -2;
-      auto grouped = [&](const std::vector<GemmPlan>& plans, void* X, int K, void* Y, int N) {
-        for (int e = 0; e < s.experts && !rc; ++e) {
-          const int start = expert_rows_host[2 * e], cnt = expert_rows_host[2 * e + 1];
-          if (cnt <= 0) continue;
-          const int bn = gemm_block_n_for(cnt);
-          CUtensorMap tm;
-          if (gemm_make_x_map(&tm, static_cast<bf16*>(X) + static_cast<size_t>(start) * K, cnt, K, K, bn)) { rc = -2; break; }
-          rc |= gemm_run(plans[e], tm, bn, static_cast<bf16*>(Y) + static_cast<size_t>(start) * N, N, cnt, st);
-          ++nl;
-        }
-      };
-      prof_start();
-      grouped(w.p_egu, hsorted, W, egu, 2 * s.ff);
-      prof_stop("moe_up");
-      const int rows = rc ? 0 : expert_rows_host[2 * (s.experts - 1)] + expert_rows_host[2 * (s.experts - 1) + 1];   // the experts' rows end here
-      KRN("glu", glu_clamped(egu, 2 * s.ff, eact, s.ff, dt, rows, s.ff, INFINITY, 1.f, st, 0.f));
-      prof_start();
-      grouped(w.p_edown, eact, s.ff, edown16, W);
-      prof_stop("moe_down");
+      if (w.il_e) {
+        KRN("moe_up", gemm_grouped_run(w.g_egu, w.xg_h, expert_rows, eact, s.ff, true, env.sms, kernel_error, st));
+      } else {
+        KRN("moe_up", gemm_grouped_run(w.g_egu, w.xg_h, expert_rows, egu, 2 * s.ff, false, env.sms, kernel_error, st));
+        KRN("glu", glu_clamped(egu, 2 * s.ff, eact, s.ff, dt, cap, s.ff, INFINITY, 1.f, st, 0.f));
+      }
+      KRN("moe_down", gemm_grouped_run(w.g_edown, w.xg_act, expert_rows, edown16, W, false, env.sms, kernel_error, st));
       KRN("moe_combine", moe_combine_add(edown16, DT_BF16, pair_pos, topw, shared_out, nullptr, 0, fo, dt, T, s.top, W, st));
       return rc;
     }
     LinearArgs up = linear_args(h, dt, w.e_gu, dt, egu, dt, cap, 2 * s.ff, W);
     up.x_rows = sorted_rows; up.tile_group = tile_group; up.wbs = gu_stride;
     KRN("moe_up", linear(up, st));
-    KRN("glu", glu_clamped(egu, 2 * s.ff, eact, s.ff, dt, cap, s.ff, INFINITY, 1.f, st, 0.f));
+    KRN("glu", glu_clamped(egu, 2 * s.ff, eact, s.ff, dt, cap, s.ff, INFINITY, 1.f, st, 0.f, w.il_e));
     LinearArgs dn = linear_args(eact, dt, w.e_down, dt, edown, DT_F32, cap, W, s.ff);
     dn.tile_group = tile_group; dn.wbs = down_stride;
     KRN("moe_down", linear(dn, st));
@@ -759,6 +761,7 @@ class Dabodra : public Model {
     const int T = b.T;
     int rc = 0;
     int64_t nl = 0;
+    if (kernel_error && *static_cast<volatile int*>(kernel_error)) { set_error("Dabodra forward: a wait inside the grouped GEMM ran out"); return -2; }
     KRN("embed", embed_normed(embed, dt, b.ids, emb_w, eps, x, h, dt, T, W, V, st));
     Pending pend;
     for (size_t li = 0; li < spec.size() && !rc; ++li) {

@@ -65,6 +65,19 @@ int gemm_run_deferred(const GemmPlan& p, const CUtensorMap& tm_x, int block_n, v
 // their head and every tile leaves through the fused epilogue `e` (epi_pass.cuh) — no fp32 segments for a consumer kernel.
 struct Gemm2Epi;
 int gemm2_run_fused(const GemmPlan& p, const CUtensorMap& tm_x, int block_n, int T, const Gemm2Epi& e, cudaStream_t st);
+// Grouped form (gemm_grouped.cu): the rows of every expert, sorted by expert, times that expert's matrix in one launch.  W: the
+// experts' [N, K] matrices stacked; expert_rows: device [experts][2] = {first row of X, rows}.  out[r, n] (leading dimension
+// ldo); with glu the rows of every matrix alternate in blocks of 64 gate rows and their 64 up rows (N % 128 == 0) and
+// out[r, i] = silu(gate_i) * up_i, i < N / 2.  N, K, ldo: multiples of 8.  error (optional, host-visible int): set to 1 when a
+// wait inside the kernel ran out.
+struct GroupedPlan {
+  CUtensorMap tm_w;
+  int experts, N, K;
+};
+int gemm_grouped_plan(GroupedPlan* p, const void* W, int experts, int N, int K);
+int gemm_grouped_x_map(CUtensorMap* tm, const void* X, int rows, int K);
+int gemm_grouped_run(const GroupedPlan& p, const CUtensorMap& tm_x, const int* expert_rows, void* out, int ldo, bool glu, int sms, int* error,
+                     cudaStream_t st);
 // Generic consumer: out[t, n] = bf16(sum of segments) — used by tests and by paths without a fused consumer.
 int reduce_partials(const PartialView& v, void* out, int ldo, int T, int N, cudaStream_t st);
 // out[t, n] (bf16, leading dimension ldo) for t < T.

@@ -79,8 +79,9 @@ int residual_dyt(float* x, const void* a, const void* f, DType ta, float mult, c
                  void* y, DType ty, const int* row_index, int rows, int W, cudaStream_t st);
 // Clamped gated unit: row t of gu (leading dimension ldgu) holds gate [F] | up [F]; g = min(gate, limit), u = clamp(up, -limit, limit),
 // y = g * sigmoid(slope * g) * (u + up_offset).  limit = INFINITY, slope = 1, up_offset = 0 is the plain SiLU-gated unit.
+// interleaved (F % 64 == 0): the row alternates in blocks of 64 gate columns and their 64 up columns instead.
 int glu_clamped(const void* gu, int ldgu, void* y, int ldy, DType t, int T, int F, float limit, float slope, cudaStream_t st,
-                float up_offset = 1.0f);
+                float up_offset = 1.0f, bool interleaved = false);
 // y[t, i] = act(y[t, i] + bias[i]) in place, i < n (leading dimension ldy; bias fp32, may be null; act: LinearAct)
 int bias_act(void* y, int ldy, const float* bias, int act, DType t, int T, int n, cudaStream_t st, float a_pos = 0.f, float a_neg = 0.f);
 // y[t, i] *= sigmoid(g[t, i]), i < n (leading dimensions ldy, ldg)

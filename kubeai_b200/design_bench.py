@@ -348,7 +348,8 @@ def _moe_roofline(z, layers, T, batch, W, kp, kd, us, hbm, tf):
         # decode: every chosen (token, expert) pair streams its expert's weights (pairs that share an expert read it from L2)
         "moe_experts_decode_frac_of_hbm": 2.0 * layers * min(batch * top, z["experts"]) * 3 * W * F / (us(kd, "moe_up") + us(kd, "moe_down")) / (hbm * 1e9),
         "shared_expert_decode_frac_of_hbm": 2.0 * layers * 3 * W * F / (us(kd, "shared_in") + us(kd, "shared_down")) / (hbm * 1e9),
-        "glu_prefill_frac_of_hbm": layers * T * (top + 1) * F * 6.0 / us(kp, "glu") / (hbm * 1e9),
+        # the gated unit as a pass of its own, where no epilogue forms it
+        **({"glu_prefill_frac_of_hbm": layers * T * (top + 1) * F * 6.0 / us(kp, "glu") / (hbm * 1e9)} if "glu" in kp else {}),
         "moe_combine_prefill_frac_of_hbm": layers * T * W * 2.0 * (top + 2) / us(kp, "moe_combine") / (hbm * 1e9),
         "moe_route_prefill_us": (us(kp, "moe_router") + us(kp, "moe_route") + us(kp, "moe_align") + us(kp, "moe_gather")) * 1e6,
     }

@@ -215,6 +215,23 @@ def test_fused_large_step_products_equal_the_plain_ones(tmp_path, monkeypatch):
     assert np.median(r) < 0.01 and np.quantile(r, 0.95) < 0.05, (np.median(r), r.max())
 
 
+@pytest.mark.parametrize("experts,top,ff,width,T", [(4, 2, 64, 72, 700), (16, 2, 192, 64, 300), (3, 1, 40, 136, 1000), (40, 8, 64, 64, 61), (8, 3, 8, 256, 33), (2, 2, 640, 264, 513), (6, 1, 128, 8, 90)])
+def test_grouped_expert_products_equal_the_plain_ones(tmp_path, monkeypatch, experts, top, ff, width, T):
+    """Experts of no, few and hundreds of rows (several row tiles), hidden sizes with the gated unit in the epilogue (multiples of
+    64) and without, partial weight tiles and k-blocks: every row is the one that the plain grouped kernels give."""
+    cfg, W, d = build(tmp_path, [delta(heads=2, kv_heads=1, dim=8, vdim=8, conv=1, mlp=moe(experts=experts, top=top, count=1, keep=1, ff=ff, shared=16))], seed=51, width=width, vocab=60,
+                      edit=lambda W: W["l0.mlp.correction"].__setitem__(slice(None), np.where(np.arange(experts) == experts - 1, -3.0, np.where(np.arange(experts) == 0, 0.4, 0.0))))
+    t = toks(T, 60, 52)
+    out = {}
+    for knob in ("1", "0"):
+        monkeypatch.setenv("B200_DB_GROUPED", knob)
+        with open_engine(d, dtype="bfloat16", max_tokens=1024, max_seqs=1) as e:
+            out[knob] = feed_whole(e, t)
+    close16(out["1"][:40], oracle_for(cfg, W).forward(t[:40]), 0.8)
+    r = rel_err(out["1"], out["0"].astype(np.float64))
+    assert np.median(r) < 0.01 and r.max() < 0.06, (np.median(r), r.max())
+
+
 @pytest.mark.parametrize("heads,kv_heads,dim,window", [(4, 2, 16, 70), (6, 1, 32, 17), (8, 8, 64, 64), (16, 1, 128, 100), (5, 5, 48, 1), (64, 1, 16, 128), (2, 1, 112, 333)])
 def test_bfloat16_tensor_core_attention_equals_the_general_kernel(tmp_path, monkeypatch, heads, kv_heads, dim, window):
     """Head sizes that fit the mma fragments, with a sink per head: the 64-row kernel against the general one on the same
