@@ -30,7 +30,6 @@
 
 #include <algorithm>
 
-#include "epi_pass.cuh"
 #include "errors.h"
 #include "gemm.h"
 #include "model.h"
@@ -121,10 +120,8 @@ class Dabodra : public Model {
   std::vector<void*> allocs;
   float* gemm_ws = nullptr;
   int* gemm_counters = nullptr;
-  int* gemm_flags = nullptr;     // of the fused form: two per CTA pair, stamped with the launch's number
-  int gemm_epoch = 0;
-  bool fuse = true;
   int few_rows = 16;
+  bool whole = true;
   CUtensorMap xm_h[kGemmNumBlockN];
   bool use_tc = false;
 
@@ -244,11 +241,6 @@ class Dabodra : public Model {
   }
 
   static int up8(int v) { return (v + 7) / 8 * 8; }
-  // a wide row is filled up to whole 256-row weight tiles (rows of zeros nobody reads), which the fused GEMM form asks for
-  static int fill_tiles(int n) {
-    const int full = (n + 255) / 256 * 256;
-    return n >= 1024 && full - n <= n / 8 ? full : n;
-  }
   void layout(LayerSpec& s) {
     int at = 0;
     auto block = [&](int* off, int n) { *off = at; at = up8(at + n); };   // every block starts 16-byte aligned
@@ -265,8 +257,8 @@ class Dabodra : public Model {
       s.conv_floats = static_cast<size_t>(std::max(s.taps, 1) - 1) * s.conv_c;
       s.rec_floats = static_cast<size_t>(s.heads) * s.dim * s.vdim;
     }
-    s.n_in = fill_tiles(at);
-    s.n_sh = s.shared ? fill_tiles(up8(2 * s.sff)) : 0;
+    s.n_in = at;
+    s.n_sh = s.shared ? up8(2 * s.sff) : 0;
   }
 
   int inspect(const CheckpointReader& ck, std::string* err) override {
@@ -343,6 +335,8 @@ class Dabodra : public Model {
       if (s.shared) rc |= mat(&w.sh_in, s.n_sh, W) | mat(&w.sh_down, W, s.sff);
     }
     if (rc) return rc;
+    if (cudaMallocHost(&kernel_error, sizeof(int)) != cudaSuccess) return -3;
+    *kernel_error = 0;
     const size_t T = e.Tcap;
     row_cap = static_cast<int>(std::min<size_t>(T, 256));
     rc |= vec(&x, T * W) | mat(&h, T, W) | mat(&inb, T, max_in) | mat(&yb, T, max_out) | mat(&ao, T, W) | mat(&hrow, row_cap, W) |
@@ -351,8 +345,6 @@ class Dabodra : public Model {
     if (max_rec) rc |= mat(&xc, T, max_xc) | vec(&o32, T * max_rec);
     if (any_moe) {
       moe_cap = static_cast<int>((T * max_top + 63) / 64 * 64) + max_e * 64;
-      if (cudaMallocHost(&kernel_error, sizeof(int)) != cudaSuccess) return -3;
-      *kernel_error = 0;
       rc |= mat(&fo, T, W) | vec(&scores, T * max_e) | vec(&topw, T * max_top) | dalloc(&topi, T * max_top * sizeof(int)) |
             dalloc(&sorted_rows, static_cast<size_t>(moe_cap) * sizeof(int)) | dalloc(&tile_group, static_cast<size_t>(moe_cap / 64) * sizeof(int)) |
             dalloc(&pair_pos, T * max_top * sizeof(int)) | mat(&egu, moe_cap, 2 * static_cast<size_t>(max_ff)) | mat(&eact, moe_cap, max_ff) |
@@ -383,9 +375,9 @@ class Dabodra : public Model {
     const size_t ws_bytes = std::max(gemm_workspace_bytes(env.sms), gemm_deferred_ws_bytes(env.sms));
     if (dalloc(&gemm_ws, ws_bytes)) return -3;
     const size_t n_counters = 2ull * (maxN / 128 + 2) * (env.Tcap / 32 + 2);
-    if (dalloc(&gemm_counters, n_counters * sizeof(int)) || dalloc(&gemm_flags, static_cast<size_t>(env.sms) * 2 * sizeof(int))) return -3;
-    if (const char* e = getenv("B200_DB_FUSE")) fuse = atoi(e) != 0;              // A/B knobs
-    if (const char* e = getenv("B200_DB_FEW_ROWS")) few_rows = atoi(e);
+    if (dalloc(&gemm_counters, n_counters * sizeof(int))) return -3;
+    if (const char* e = getenv("B200_DB_FEW_ROWS")) few_rows = atoi(e);            // A/B knobs
+    if (const char* e = getenv("B200_DB_WHOLE")) whole = atoi(e) != 0;
     bool grouped = true;
     if (const char* e = getenv("B200_DB_GROUPED")) grouped = atoi(e) != 0;
     const int bns[kGemmNumBlockN] = {32, 64, 128, 256, 512};
@@ -579,39 +571,23 @@ class Dabodra : public Model {
   }
 
   // ------------------------------------------------------------ forward
-  // Y = X W^T.  Steps of up to 16 tokens stream the weights through linear.cu's fragment kernel.  Larger steps take the pair
-  // GEMM, in its fused form (whole 256-row tiles, at least one tile per CTA pair) or in its plain one.
-  bool takes_fused(const GemmPlan& plan, bool tc, int T, int N) const {
-    const int bn = block_n(plan, T);
-    return tc && T > few_rows && fuse && N % 256 == 0 && T > 128 && N / 256 * ((T + bn - 1) / bn) >= plan.max_ctas / 2;
-  }
-  int run_fused(const GemmPlan& plan, const CUtensorMap* xm, int epi, void* Y, int ldy, int T) {
-    const int bn = block_n(plan, T);
-    Gemm2Epi e;
-    memset(&e, 0, sizeof(e));
-    e.epi = epi;
-    e.out = static_cast<bf16*>(Y); e.ldo = ldy;
-    e.flags = gemm_flags; e.epoch = ++gemm_epoch;
-    return gemm2_run_fused(plan, xm[gemm_block_n_index(bn)], bn, T, e, env.stream);
+  // Y = X W^T.  Steps of up to 16 tokens stream the weights through linear.cu's fragment kernel, steps of up to 256 tokens take
+  // the stream-K pair GEMM (every weight byte once, all pairs busy), larger ones whole tiles.
+  // The grouped kernel on one matrix: whole 256 x 256 tiles, the accumulator drained under the next tile.
+  bool takes_whole(bool tc, int T) const { return tc && T > 256 && whole; }
+  int run_whole(const GemmPlan& plan, const CUtensorMap* xm, bool glu, void* Y, int ldy, int T) {
+    GroupedPlan g;
+    g.tm_w = plan.tm_w; g.experts = 1; g.N = plan.N; g.K = plan.K;      // the same boxes: 128 rows x 64 columns on both sides
+    return gemm_grouped_run(g, xm[gemm_block_n_index(256)], nullptr, Y, ldy, glu, env.sms, kernel_error, env.stream, T);
   }
   int project(const GemmPlan& plan, bool tc, const CUtensorMap* xm, const void* X, const void* Wm, void* Y, int T, int N, int K) {
+    if (takes_whole(tc, T)) return run_whole(plan, xm, false, Y, N, T);
     if (tc && T > few_rows) {
-      if (takes_fused(plan, tc, T, N)) return run_fused(plan, xm, GEMM3_EPI_PLAIN, Y, N, T);
-      const int bn = block_n(plan, T);
+      const int bn = gemm_block_n_for(T);
       return gemm_run(plan, xm[gemm_block_n_index(bn)], bn, Y, N, T, env.stream);
     }
     return linear(linear_args(X, dt, Wm, dt, Y, dt, T, N, K), env.stream);
   }
-  // Token-tile size: where 512-token tiles neither fill the pairs nor are close enough to one whole tile per pair (that form
-  // takes up to 64 k-blocks), 256-token tiles give the fused form its tile per pair.
-  int block_n(const GemmPlan& p, int T) const {
-    const int bn = gemm_block_n_for(T), pairs = p.max_ctas / 2;
-    if (bn != 512 || !fuse || p.N % 256) return bn;
-    const int t512 = p.N / 256 * ((T + 511) / 512), t256 = p.N / 256 * ((T + 255) / 256);
-    const bool whole = p.K <= 4096 && t512 * 5 >= pairs * 3;
-    return t512 < pairs && !whole && t256 >= pairs ? 256 : bn;
-  }
-
   // per-kernel device time (b200_engine_kernel_times): with profiling on, every launch is bracketed by events and waited for
   cudaEvent_t pe0 = nullptr, pe1 = nullptr;
   void prof_start() {
@@ -705,8 +681,8 @@ class Dabodra : public Model {
     KRN("moe_route", moe_route(scores, topi, topw, T, s.experts, s.groups, s.keep, s.top, st, MOE_SIGMOID, s.experts, w.correction, form));
     const void* shared_out = nullptr;
     if (s.shared) {
-      if (w.il_s && s.n_sh == 2 * s.sff && takes_fused(w.p_shin, w.tc_shin, T, s.n_sh)) {
-        KRN("shared_in", run_fused(w.p_shin, xm_h, GEMM3_EPI_SILU, shact, s.sff, T));     // the gated unit in the epilogue
+      if (w.il_s && takes_whole(w.tc_shin, T)) {
+        KRN("shared_in", run_whole(w.p_shin, xm_h, true, shact, s.sff, T));     // the gated unit in the epilogue
       } else {
         KRN("shared_in", project(w.p_shin, w.tc_shin, xm_h, h, w.sh_in, sh, T, s.n_sh, W));
         KRN("glu", glu_clamped(sh, s.n_sh, shact, s.sff, dt, T, s.sff, INFINITY, 1.f, st, 0.f, w.il_s));

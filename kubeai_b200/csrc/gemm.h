@@ -69,7 +69,7 @@ int gemm2_run_fused(const GemmPlan& p, const CUtensorMap& tm_x, int block_n, int
 // experts' [N, K] matrices stacked; expert_rows: device [experts][2] = {first row of X, rows}.  out[r, n] (leading dimension
 // ldo); with glu the rows of every matrix alternate in blocks of 64 gate rows and their 64 up rows (N % 128 == 0) and
 // out[r, i] = silu(gate_i) * up_i, i < N / 2.  N, K, ldo: multiples of 8.  error (optional, host-visible int): set to 1 when a
-// wait inside the kernel ran out.
+// wait inside the kernel ran out.  expert_rows may be null for one matrix and `rows` rows: a plain product in whole tiles.
 struct GroupedPlan {
   CUtensorMap tm_w;
   int experts, N, K;
@@ -77,7 +77,7 @@ struct GroupedPlan {
 int gemm_grouped_plan(GroupedPlan* p, const void* W, int experts, int N, int K);
 int gemm_grouped_x_map(CUtensorMap* tm, const void* X, int rows, int K);
 int gemm_grouped_run(const GroupedPlan& p, const CUtensorMap& tm_x, const int* expert_rows, void* out, int ldo, bool glu, int sms, int* error,
-                     cudaStream_t st);
+                     cudaStream_t st, int rows = 0);
 // Generic consumer: out[t, n] = bf16(sum of segments) — used by tests and by paths without a fused consumer.
 int reduce_partials(const PartialView& v, void* out, int ldo, int T, int N, cudaStream_t st);
 // out[t, n] (bf16, leading dimension ldo) for t < T.

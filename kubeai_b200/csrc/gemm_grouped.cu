@@ -47,12 +47,12 @@ struct Tile {
 // Walks this pair's items: `next` advances by one item of the pair, expert by expert.
 struct Walk {
   const int* expert_rows;
-  int experts, mt, N;
+  int experts, mt, N, rows;   // without a table: one matrix, `rows` rows from 0
   int e = 0;
   long long base = 0;    // items of the experts before e
   __device__ bool at(long long item, Tile* t) {
     while (e < experts) {
-      const int cnt = expert_rows[2 * e + 1];
+      const int cnt = expert_rows ? expert_rows[2 * e + 1] : rows;
       const int ntt = (cnt + kRows - 1) / kRows;
       const long long n = static_cast<long long>(ntt) * mt;
       if (item < base + n) {
@@ -60,7 +60,7 @@ struct Walk {
         const int per = ((cnt + ntt - 1) / ntt + 15) & ~15;     // equal tiles, whole 16-row steps (at most kRows)
         t->n0 = m * 2 * kSlab;
         t->wrow = e * N + t->n0;
-        t->row0 = expert_rows[2 * e] + tt * per;
+        t->row0 = (expert_rows ? expert_rows[2 * e] : 0) + tt * per;
         t->rows = min(per, cnt - tt * per);
         if (t->rows > 0) return true;
         t->rows = 0;       // rounding up to 16 may leave the last tile of an expert empty
@@ -95,7 +95,7 @@ __device__ __forceinline__ bool all_epilogue(bool v) {
 }
 
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(kThreads, 1)
-gemm_grouped_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__ CUtensorMap tm_x, const int* expert_rows, int experts,
+gemm_grouped_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__ CUtensorMap tm_x, const int* expert_rows, int experts, int rows,
                     bf16* out, int ldo, int N, int K, int glu, int* error) {
   extern __shared__ uint8_t smem_raw[];
   const uint32_t smem_base = (smem_u32(smem_raw) + 1023u) & ~1023u;
@@ -111,7 +111,7 @@ gemm_grouped_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_const
   const bool leader = rank == 0;
   const int units = gridDim.x >> 1, unit = blockIdx.x >> 1, KB = (K + kBlockK - 1) / kBlockK;
   Walk walk;
-  walk.expert_rows = expert_rows; walk.experts = experts; walk.mt = (N + 2 * kSlab - 1) / (2 * kSlab); walk.N = N;
+  walk.expert_rows = expert_rows; walk.experts = experts; walk.mt = (N + 2 * kSlab - 1) / (2 * kSlab); walk.N = N; walk.rows = rows;
 
   if (warp == 0 && lane == 0) {
     tma_prefetch_desc(&tm_w);
@@ -262,11 +262,11 @@ int gemm_grouped_plan(GroupedPlan* p, const void* W, int experts, int N, int K) 
 int gemm_grouped_x_map(CUtensorMap* tm, const void* X, int rows, int K) { return tmap_encode_bf16_2d(tm, X, rows, K, K, kRows / 2, kBlockK, 1); }
 
 int gemm_grouped_run(const GroupedPlan& p, const CUtensorMap& tm_x, const int* expert_rows, void* out, int ldo, bool glu, int sms, int* error,
-                     cudaStream_t st) {
-  if (!expert_rows || !out || ldo % 8 || reinterpret_cast<uintptr_t>(out) % 16 || sms < 2 || (glu && p.N % kSlab)) return -1;
+                     cudaStream_t st, int rows) {
+  if ((!expert_rows && (p.experts != 1 || rows < 1)) || !out || ldo % 8 || reinterpret_cast<uintptr_t>(out) % 16 || sms < 2 || (glu && p.N % kSlab)) return -1;
   static std::atomic<unsigned long long> attr{0};
   if (!ensure_dynamic_smem(gemm_grouped_kernel, kSmem, &attr)) return -2;
-  gemm_grouped_kernel<<<sms / 2 * 2, kThreads, kSmem, st>>>(p.tm_w, tm_x, expert_rows, p.experts, static_cast<bf16*>(out), ldo, p.N, p.K, glu ? 1 : 0, error);
+  gemm_grouped_kernel<<<sms / 2 * 2, kThreads, kSmem, st>>>(p.tm_w, tm_x, expert_rows, p.experts, rows, static_cast<bf16*>(out), ldo, p.N, p.K, glu ? 1 : 0, error);
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
 

@@ -334,6 +334,47 @@ __device__ __forceinline__ void stf4(bf16* p, float4 v) {
   const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
   *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
 }
+// The per-head output stage for whole fours of columns: a warp per (token, head), the head's row in registers.
+template <typename T, int NF>
+__global__ void __launch_bounds__(128) out_gate_vec_kernel(OutGateArgs a, long long units) {
+  const int lane = threadIdx.x & 31;
+  const long long p = static_cast<long long>(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (p >= units) return;
+  const long long t = p / a.heads;
+  const int c0 = static_cast<int>(p - t * a.heads) * a.vdim;
+  const float* op = a.o + p * a.vdim;
+  const T* g = a.g ? static_cast<const T*>(a.g) + t * a.ldg + c0 : nullptr;
+  const float* w = a.w ? a.w + (a.w_full ? c0 : 0) : nullptr;
+  T* y = static_cast<T*>(a.y) + t * a.ldy + c0;
+  const float dinv = a.den_nq ? 1.0f / (fmaxf(fabsf(a.den_nq[p]), a.den_floor[p]) + a.den_eps) : 1.0f;
+  float4 v[NF], gv[NF];
+  float ss = 0.f;
+#pragma unroll
+  for (int f = 0; f < NF; ++f) {
+    const int i = (lane + 32 * f) * 4;
+    if (i < a.vdim) {
+      v[f] = ldf4(op + i);
+      if (g) gv[f] = ldf4(g + i);
+      v[f].x *= dinv; v[f].y *= dinv; v[f].z *= dinv; v[f].w *= dinv;
+      ss = fmaf(v[f].x, v[f].x, ss); ss = fmaf(v[f].y, v[f].y, ss); ss = fmaf(v[f].z, v[f].z, ss); ss = fmaf(v[f].w, v[f].w, ss);
+    }
+  }
+  for (int s = 16; s > 0; s >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, s);
+  const float inv = 1.0f / sqrtf(ss / static_cast<float>(a.vdim) + a.eps);
+  auto gate_of = [&](float z) { const float sg = 1.0f / (1.0f + expf(-z)); return a.gate_act == GATE_SIGMOID ? sg : z * sg; };
+#pragma unroll
+  for (int f = 0; f < NF; ++f) {
+    const int i = (lane + 32 * f) * 4;
+    if (i < a.vdim) {
+      const float4 ww = w ? ldf4(w + i) : make_float4(1.f, 1.f, 1.f, 1.f);
+      float4 gt = make_float4(1.f, 1.f, 1.f, 1.f);
+      if (g) gt = make_float4(gate_of(gv[f].x), gate_of(gv[f].y), gate_of(gv[f].z), gate_of(gv[f].w));
+      stf4(y + i, make_float4(v[f].x * inv * ww.x * gt.x * a.out_scale, v[f].y * inv * ww.y * gt.y * a.out_scale, v[f].z * inv * ww.z * gt.z * a.out_scale,
+                              v[f].w * inv * ww.w * gt.w * a.out_scale));
+    }
+  }
+}
+
 template <typename T, bool VEC>
 __global__ void __launch_bounds__(256) gated_group_norm_kernel(GatedGroupNormArgs a) {
   extern __shared__ __align__(16) float us[];
@@ -458,6 +499,16 @@ int recurrent_out_gate(const OutGateArgs& a, cudaStream_t st) {
   if (!a.o || !a.y || a.heads < 1 || a.vdim < 1) return -1;
   if (a.joint && (a.w_full || a.den_nq)) return -1;
   if (a.den_nq && !a.den_floor) return -1;
+  auto al16 = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+  if (!a.joint && a.vdim % 4 == 0 && a.vdim <= 256 && a.ldg % 4 == 0 && a.ldy % 4 == 0 && al16(a.o) && al16(a.g) && al16(a.y) && al16(a.w)) {
+    const unsigned ctas = static_cast<unsigned>((units + 3) / 4);
+    if (a.t == DT_BF16) {
+      if (a.vdim <= 128) out_gate_vec_kernel<bf16, 1><<<ctas, 128, 0, st>>>(a, units); else out_gate_vec_kernel<bf16, 2><<<ctas, 128, 0, st>>>(a, units);
+    } else {
+      if (a.vdim <= 128) out_gate_vec_kernel<float, 1><<<ctas, 128, 0, st>>>(a, units); else out_gate_vec_kernel<float, 2><<<ctas, 128, 0, st>>>(a, units);
+    }
+    return cudaGetLastError() == cudaSuccess ? 0 : -2;
+  }
   const int th = a.joint ? (a.heads * a.vdim >= 1024 ? 256 : 128) : 128;
   const unsigned grid = static_cast<unsigned>(a.joint ? units : (units + 3) / 4);
   if (a.t == DT_BF16) recurrent_out_gate_kernel<bf16><<<grid, th, 0, st>>>(a, units);

@@ -8,7 +8,8 @@
 // products; either way one output element is accumulated in an order that does not depend on what else is in the batch), and
 // two kernels for the few rows of a decode step: up to 16 rows of a bf16 matrix whose rows are whole 16-byte pieces go through
 // mma.sync with the weights as the 16-row operand (every weight byte is loaded once, straight into fragments), anything else of
-// up to 8 rows through one warp per output row.
+// up to 8 rows through one warp per output row.  Many rows against up to 64 columns take the fragment kernel with the operands
+// exchanged.
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <stdlib.h>
@@ -296,7 +297,10 @@ __device__ __forceinline__ uint4 ldx8(const float* p, uint4* lo) {
   return make_uint4(h[0], h[1], h[2], h[3]);
 }
 
-template <typename TX, typename TY, int NB, int U>
+// THIN: the same with the operands' parts exchanged, for many rows of X against few rows of W (router logits, scalar gates):
+// X streams as the 16-row operand, W's rows 16 y .. 16 y + 15 of grid row y are the "tokens".  One output element is summed in
+// the same order as above.
+template <typename TX, typename TY, int NB, int U, bool THIN>
 __global__ void __launch_bounds__(256) linear_rows_mma_kernel(LinearArgs a, int KS) {
   constexpr bool SPLIT = sizeof(TX) == 4;
   __shared__ float part[8][16][8 * NB + 1];   // [warp][weight row][token]
@@ -304,16 +308,19 @@ __global__ void __launch_bounds__(256) linear_rows_mma_kernel(LinearArgs a, int 
   const int ks = wrp % KS, RG = 8 / KS;
   const int n0 = (blockIdx.x * RG + wrp / KS) * 16;
   const long long b = blockIdx.z;
-  const bf16* W = static_cast<const bf16*>(a.W) + b * a.wbs;
-  const TX* X = static_cast<const TX*>(a.X) + b * a.xbs;
+  const int col0 = THIN ? blockIdx.y * 8 * NB : 0;
+  // the 16-row operand and its rows, the 8-row operand and its rows
+  const bf16* W = THIN ? static_cast<const bf16*>(a.X) : static_cast<const bf16*>(a.W) + b * a.wbs;
+  const TX* X = THIN ? static_cast<const TX*>(a.W) + static_cast<long long>(col0) * a.ldw : static_cast<const TX*>(a.X) + b * a.xbs;
+  const int ldw = THIN ? a.ldx : a.ldw, ldx = THIN ? a.ldw : a.ldx, rows = THIN ? a.T : a.N, toks = THIN ? min(8 * NB, a.N - col0) : a.T;
   TY* Y = static_cast<TY*>(a.Y) + b * a.ybs;
-  const bool r0 = n0 + g < a.N, r1 = n0 + g + 8 < a.N;
-  const bf16* w0 = W + static_cast<long long>(n0 + g) * a.ldw;
-  const bf16* w1 = w0 + 8ll * a.ldw;
+  const bool r0 = n0 + g < rows, r1 = n0 + g + 8 < rows;
+  const bf16* w0 = W + static_cast<long long>(n0 + g) * ldw;
+  const bf16* w1 = w0 + 8ll * ldw;
   const TX* xr[NB];
   bool xin[NB];
 #pragma unroll
-  for (int i = 0; i < NB; ++i) { xin[i] = g + 8 * i < a.T; xr[i] = X + static_cast<long long>(g + 8 * i) * a.ldx; }
+  for (int i = 0; i < NB; ++i) { xin[i] = g + 8 * i < toks; xr[i] = X + static_cast<long long>(g + 8 * i) * ldx; }
   float acc[NB][4];
 #pragma unroll
   for (int i = 0; i < NB; ++i)
@@ -361,10 +368,11 @@ __global__ void __launch_bounds__(256) linear_rows_mma_kernel(LinearArgs a, int 
   for (int e = threadIdx.x; e < RG * 16 * 8 * NB; e += 256) {
     const int r = e % (RG * 16), t = e / (RG * 16), rg = r >> 4;     // neighbouring threads: neighbouring output columns
     const int n = blockIdx.x * RG * 16 + r;
-    if (t >= a.T || n >= a.N) continue;
+    if (t >= toks || n >= rows) continue;
     float v = 0.f;
     for (int k = 0; k < KS; ++k) v += part[rg * KS + k][r & 15][t];
-    st1(Y + static_cast<long long>(t) * a.ldy + n, finish<TY>(a, a.row_scale ? v * a.row_scale[t] : v, n));
+    const int yr = THIN ? n : t, yc = THIN ? col0 + t : n;
+    st1(Y + static_cast<long long>(yr) * a.ldy + yc, finish<TY>(a, a.row_scale ? v * a.row_scale[yr] : v, yc));
   }
 }
 
@@ -416,9 +424,20 @@ int launch_linear(const LinearArgs& a, cudaStream_t st) {
       const int KS = steps >= 32 ? 8 : (steps >= 16 ? 4 : (steps >= 8 ? 2 : 1));
       dim3 grid((a.N + 128 / KS - 1) / (128 / KS), 1, a.batch);
       constexpr int U = sizeof(TX) == 4 ? 4 : 8;
-      if (a.T <= 8) linear_rows_mma_kernel<TX, TY, 1, U><<<grid, 256, 0, st>>>(a, KS);
-      else linear_rows_mma_kernel<TX, TY, 2, U / 2><<<grid, 256, 0, st>>>(a, KS);
+      if (a.T <= 8) linear_rows_mma_kernel<TX, TY, 1, U, false><<<grid, 256, 0, st>>>(a, KS);
+      else linear_rows_mma_kernel<TX, TY, 2, U / 2, false><<<grid, 256, 0, st>>>(a, KS);
       return cudaGetLastError() == cudaSuccess ? 0 : -2;
+    }
+    if constexpr (sizeof(TX) == 2) {
+      // B200_LIN_THIN: A/B knob, the most columns that take the exchanged form (0: none)
+      static const int thin = [] { const char* e = getenv("B200_LIN_THIN"); return e ? atoi(e) : 64; }();
+      if (vec && a.N <= thin && a.batch == 1 && !a.x_rows && !a.tile_group) {
+        const int steps = (a.K + 31) / 32;
+        const int KS = steps >= 32 ? 8 : (steps >= 16 ? 4 : (steps >= 8 ? 2 : 1));
+        dim3 grid((a.T + 128 / KS - 1) / (128 / KS), (a.N + 15) / 16);
+        linear_rows_mma_kernel<TX, TY, 2, 4, true><<<grid, 256, 0, st>>>(a, KS);
+        return cudaGetLastError() == cudaSuccess ? 0 : -2;
+      }
     }
   }
   if (few) {

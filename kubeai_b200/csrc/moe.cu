@@ -166,6 +166,35 @@ __global__ void moe_combine_kernel(const TYIN* y, const int* pair_pos, const flo
   }
 }
 
+// bf16 rows of whole 16-byte pieces: a thread forms eight neighbouring columns, the same sums in the same order
+__global__ void __launch_bounds__(256) moe_combine_vec_kernel(const bf16* y, const int* pair_pos, const float* topk_w, bf16* out, int top, int W, const bf16* add,
+                                                              const float* add_gate, int ld_gate) {
+  const long long t = blockIdx.x;
+  const float gate = add && add_gate ? 1.0f / (1.0f + expf(-add_gate[t * ld_gate])) : 1.f;
+  auto fma8 = [](float* acc, float s, const bf16* p) {
+    const uint4 r = *reinterpret_cast<const uint4*>(p);
+    const uint32_t u[4] = {r.x, r.y, r.z, r.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      acc[2 * i] = fmaf(s, __uint_as_float(u[i] << 16), acc[2 * i]);
+      acc[2 * i + 1] = fmaf(s, __uint_as_float(u[i] & 0xffff0000u), acc[2 * i + 1]);
+    }
+  };
+  for (int i = threadIdx.x * 8; i < W; i += blockDim.x * 8) {
+    float acc[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+#pragma unroll 4
+    for (int k = 0; k < top; ++k) fma8(acc, topk_w ? topk_w[t * top + k] : 1.f, y + static_cast<long long>(pair_pos[t * top + k]) * W + i);
+    if (add) fma8(acc, gate, add + t * W + i);
+    uint32_t o[4];
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const __nv_bfloat162 b = __floats2bfloat162_rn(acc[2 * k], acc[2 * k + 1]);
+      o[k] = *reinterpret_cast<const uint32_t*>(&b);
+    }
+    *reinterpret_cast<uint4*>(out + t * W + i) = make_uint4(o[0], o[1], o[2], o[3]);
+  }
+}
+
 }  // namespace
 
 int moe_route(float* scores, int* topk_ids, float* topk_w, int T, int E, int groups, int keep, int top, cudaStream_t st, int score_fn, int ld,
@@ -204,7 +233,11 @@ int moe_combine_add(const void* y, DType ty, const int* pair_pos, const float* t
   if (T <= 0) return 0;
   if (!y || !pair_pos || !out || top < 1 || (ty == DT_BF16 && t != DT_BF16)) return -1;
   const int th = W >= 1024 ? 256 : 128;
-  if (ty == DT_BF16)
+  auto al16 = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+  if (ty == DT_BF16 && W % 8 == 0 && al16(y) && al16(out) && al16(add))
+    moe_combine_vec_kernel<<<T, W >= 2048 ? 256 : 128, 0, st>>>(static_cast<const bf16*>(y), pair_pos, topk_w, static_cast<bf16*>(out), top, W,
+                                                                static_cast<const bf16*>(add), add_gate, ld_gate);
+  else if (ty == DT_BF16)
     moe_combine_kernel<bf16, bf16><<<T, th, 0, st>>>(static_cast<const bf16*>(y), pair_pos, topk_w, static_cast<bf16*>(out), top, W,
                                                        static_cast<const bf16*>(add), add_gate, ld_gate);
   else if (t == DT_BF16)

@@ -97,7 +97,12 @@ __global__ void __launch_bounds__(128) short_conv_vec_kernel(ShortConvArgs a, in
   for (int e = 0; e < VEC; ++e) {
     bias[e] = a.bias ? a.bias[c + e] : 0.f;
 #pragma unroll
-    for (int j = 0; j < TAPS; ++j) w[j][e] = a.w[static_cast<long long>(c + e) * TAPS + j];
+    for (int j = 0; j < TAPS; ++j)
+      if (TAPS != 4) w[j][e] = a.w[static_cast<long long>(c + e) * TAPS + j];
+    if constexpr (TAPS == 4) {
+      const float4 q = *reinterpret_cast<const float4*>(a.w + static_cast<long long>(c + e) * 4);
+      w[0][e] = q.x; w[1][e] = q.y; w[2][e] = q.z; w[3][e] = q.w;
+    }
   }
   int cur = -1;
   for (long long t = t0; t < t1; ++t) {
@@ -135,7 +140,8 @@ __global__ void __launch_bounds__(128) short_conv_vec_kernel(ShortConvArgs a, in
 #pragma unroll
       for (int k = 0; k < TAPS - 1; ++k) r = fmaf(w[k][e], hist[k][e], r);     // oldest tap first, the token's own last
       r = fmaf(w[TAPS - 1][e], v[e], r);
-      acc[e] = a.act == CONV_SILU ? siluf_(r) : r;
+      // an output that is rounded to bf16 takes the fast exponential and division
+      acc[e] = a.act == CONV_SILU ? (VEC == 8 ? __fdividef(r, 1.0f + __expf(-r)) : siluf_(r)) : r;
     }
 #pragma unroll
     for (int k = 0; k + 1 < TAPS - 1; ++k)
@@ -261,7 +267,7 @@ int short_conv(const ShortConvArgs& a, cudaStream_t st) {
   const long long total = static_cast<long long>(a.T) * a.C;
   const int vec = a.t == DT_BF16 ? 8 : 4;
   if (a.t == a.ty && a.taps >= 1 && a.taps <= 4 && a.C % vec == 0 && a.ldu % vec == 0 && a.ldy % vec == 0 && reinterpret_cast<uintptr_t>(a.u) % 16 == 0 &&
-      reinterpret_cast<uintptr_t>(a.y) % 16 == 0) {
+      reinterpret_cast<uintptr_t>(a.y) % 16 == 0 && reinterpret_cast<uintptr_t>(a.w) % 16 == 0) {
     // rows per walk: long enough to amortise the window's fill, short enough to leave every SM several CTAs
     const int groups = a.C / vec;
     int TB = 16;

@@ -195,6 +195,71 @@ __global__ void __launch_bounds__(1024) conv_qk_prep_kernel(ConvQkPrepArgs a) {
   }
 }
 
+// The same without a convolution, for bf16 rows of whole 16-byte pieces and neighbouring rotation pairs: a thread owns eight
+// columns of the query or key row from the load to the store, so only the two sums go through shared memory.
+__global__ void __launch_bounds__(1024) qk_rows_prep_kernel(ConvQkPrepArgs a) {
+  __shared__ float red[2][32];
+  const long long t = blockIdx.x;
+  const int lane = threadIdx.x & 31, wrp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  const int D = a.dim, HD = a.heads * D, GD = a.kv_heads * D, C = HD + GD, c0 = threadIdx.x * 8;
+  const bool in = c0 < C, isq = c0 < HD;
+  bf16* cache = static_cast<bf16*>(a.cache) + static_cast<long long>(a.slots[t]) * (2ll * GD);
+  float v[8];
+  float ss = 0.f;
+  if (in) {
+    const uint4 r = *reinterpret_cast<const uint4*>(static_cast<const bf16*>(a.qk) + t * a.ld + c0);
+    if (!isq) *reinterpret_cast<uint4*>(cache + GD + (c0 - HD)) = r;      // the values
+    const uint32_t u[4] = {r.x, r.y, r.z, r.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      v[2 * i] = __uint_as_float(u[i] << 16);
+      v[2 * i + 1] = __uint_as_float(u[i] & 0xffff0000u);
+      ss = fmaf(v[2 * i], v[2 * i], ss);
+      ss = fmaf(v[2 * i + 1], v[2 * i + 1], ss);
+    }
+  }
+  float sq = in && isq ? ss : 0.f, sk = in && !isq ? ss : 0.f;
+  for (int o = 16; o > 0; o >>= 1) { sq += __shfl_xor_sync(0xffffffffu, sq, o); sk += __shfl_xor_sync(0xffffffffu, sk, o); }
+  if (lane == 0) { red[0][wrp] = sq; red[1][wrp] = sk; }
+  __syncthreads();
+  if (!in) return;
+  float tot = 0.f;
+  for (int w = 0; w < nw; ++w) tot += red[isq ? 0 : 1][w];
+  const float inv = 1.0f / sqrtf(tot / static_cast<float>(isq ? HD : GD) + a.eps);
+  const int cc = isq ? c0 : c0 - HD, d0 = cc % D;
+  const float* nwt = isq ? a.q_norm_w : a.k_norm_w;
+  if (nwt) {
+    const float4 w0 = *reinterpret_cast<const float4*>(nwt + cc), w1 = *reinterpret_cast<const float4*>(nwt + cc + 4);
+    const float w[8] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v[i] = v[i] * inv * w[i];
+  } else {
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v[i] *= inv;
+  }
+  const int half = a.rot_dims / 2;
+  const float2* cs = half ? a.rope + static_cast<long long>(a.positions[t]) * half + d0 / 2 : nullptr;
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+    if (d0 / 2 + i < half) {
+      const float2 r = cs[i];
+      const float x0 = v[2 * i], x1 = v[2 * i + 1];
+      v[2 * i] = x0 * r.x - x1 * r.y;
+      v[2 * i + 1] = x1 * r.x + x0 * r.y;
+    }
+  if (isq) {
+    const float hs = a.q_head_scale ? a.q_head_scale[cc / D] : 1.0f;
+    float4* dst = reinterpret_cast<float4*>(a.qn + t * HD + cc);
+    dst[0] = make_float4(v[0] * hs, v[1] * hs, v[2] * hs, v[3] * hs);
+    dst[1] = make_float4(v[4] * hs, v[5] * hs, v[6] * hs, v[7] * hs);
+  } else {
+    uint32_t o[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) { const __nv_bfloat162 b = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]); o[i] = *reinterpret_cast<const uint32_t*>(&b); }
+    *reinterpret_cast<uint4*>(cache + cc) = make_uint4(o[0], o[1], o[2], o[3]);
+  }
+}
+
 // ---------------------------------------------------------------------------------------------- attention, any head size
 constexpr int kWarps = 4, kWarpsDecode = 16;
 constexpr int kMaxVR = 8;   // value columns per lane: vdim <= 256
@@ -653,6 +718,12 @@ int conv_qk_prep(const ConvQkPrepArgs& a, cudaStream_t st) {
   if (smem > 200 * 1024) return -1;
   // steps of few tokens leave most SMs idle, so a token's CTA is as wide as its row allows (a thread per channel up to the
   // CTA's limit); steps of many tokens keep more CTAs per SM with narrower ones
+  auto al16 = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+  if (a.t == DT_BF16 && !a.conv_w && (a.interleaved || !a.rot_dims) && a.dim % 8 == 0 && a.ld % 8 == 0 && C <= 8192 && al16(a.qk) && al16(a.cache) && al16(a.qn) &&
+      al16(a.q_norm_w) && al16(a.k_norm_w)) {
+    qk_rows_prep_kernel<<<a.T, (C / 8 + 31) / 32 * 32, 0, st>>>(a);
+    return cudaGetLastError() == cudaSuccess ? 0 : -2;
+  }
   const int th = a.T >= 256 ? (C >= 2048 ? 256 : 128) : std::min(1024, std::max(128, (C + 31) / 32 * 32));
   if (a.t == DT_BF16) {
     if (smem > 48 * 1024 && !ensure_dynamic_smem(conv_qk_prep_kernel<bf16>, 200 * 1024, &set16)) return -2;

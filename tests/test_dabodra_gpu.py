@@ -196,10 +196,10 @@ def test_medium_sizes_on_every_projection_and_expert_path(tmp_path, dtype):
     check(parts, want)
 
 
-def test_fused_large_step_products_equal_the_plain_ones(tmp_path, monkeypatch):
-    """Matrices of whole 256-row tiles in a step with a tile per CTA pair and more take the fused GEMM form (the filled-up
-    input projection, the shared expert); the step's last token tiles are partial.  All rows are those of the plain form."""
-    layers = [attention(heads=16, kv_heads=4, dim=64, window=300, rot_dims=32, scale=0.125, mlp=moe(experts=2, top=1, count=1, keep=1, ff=64, shared=2048)),
+def test_whole_tile_products_of_large_steps_equal_the_stream_k_ones(tmp_path, monkeypatch):
+    """Steps of more than 256 tokens take whole-tile products, the shared expert with its gated unit in the epilogue; the last
+    token tiles and the last weight tiles are partial.  All rows are those of the stream-K form with a pass of its own."""
+    layers = [attention(heads=16, kv_heads=4, dim=64, window=300, rot_dims=32, scale=0.125, mlp=moe(experts=2, top=1, count=1, keep=1, ff=64, shared=1984)),
               delta(heads=8, kv_heads=4, dim=96, vdim=120, conv=4, mlp=None)]
     cfg, W, d = build(tmp_path, layers, seed=81, width=2048, vocab=64)
     T = 4700
@@ -207,7 +207,7 @@ def test_fused_large_step_products_equal_the_plain_ones(tmp_path, monkeypatch):
     rows = sorted(set(range(24)) | set(range(100, T, 97)) | {255, 256, 511, 512, 4095, 4096, 4607, 4608, T - 1})
     out = {}
     for knob in ("1", "0"):
-        monkeypatch.setenv("B200_DB_FUSE", knob)
+        monkeypatch.setenv("B200_DB_WHOLE", knob)
         with open_engine(d, dtype="bfloat16", max_tokens=4704, max_seqs=1) as e:
             out[knob] = feed_whole(e, t, rows)
     close16(out["1"][:24], oracle_for(cfg, W).forward(t[:24]))
