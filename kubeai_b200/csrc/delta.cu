@@ -51,13 +51,15 @@ __global__ void __launch_bounds__(kThreads) delta_scan_kernel(DeltaArgs a, int P
   float* Sg = a.states + (static_cast<long long>(slot) * a.heads + head) * D * Dv + j;
   const bool live = j < Dv;
   float S[kPieces][4];
+  {
+    const float* r = Sg + static_cast<long long>(4 * p) * Dv;      // one pointer walks the lane's rows
+    const long long skip = static_cast<long long>(4 * P - 4) * Dv;
+    const bool held = live && pos0 > 0;
 #pragma unroll
-  for (int m = 0; m < kPieces; ++m)
+    for (int m = 0; m < kPieces; ++m, r += skip)
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int i = 4 * (m * P + p) + e;
-      S[m][e] = (live && m < M && i < D && pos0 > 0) ? Sg[static_cast<long long>(i) * Dv] : 0.f;
-    }
+      for (int e = 0; e < 4; ++e, r += Dv) S[m][e] = (held && m < M && 4 * (m * P + p) + e < D) ? *r : 0.f;
+  }
   const float rate = a.rate[head], dt_bias = a.dt_bias[head];
   for (int g0 = 0; g0 < n; g0 += G) {
     const int gn = min(G, n - g0);
@@ -135,13 +137,13 @@ __global__ void __launch_bounds__(kThreads) delta_scan_kernel(DeltaArgs a, int P
     }
   }
   if (live) {
+    float* r = Sg + static_cast<long long>(4 * p) * Dv;
+    const long long skip = static_cast<long long>(4 * P - 4) * Dv;
 #pragma unroll
-    for (int m = 0; m < kPieces; ++m)
+    for (int m = 0; m < kPieces; ++m, r += skip)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int i = 4 * (m * P + p) + e;
-        if (m < M && i < D) Sg[static_cast<long long>(i) * Dv] = S[m][e];
-      }
+      for (int e = 0; e < 4; ++e, r += Dv)
+        if (m < M && 4 * (m * P + p) + e < D) *r = S[m][e];
   }
 }
 
